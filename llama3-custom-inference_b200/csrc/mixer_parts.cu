@@ -1,0 +1,251 @@
+// The memory-bound steps around the mixers of a decoder with a 32-bit residual stream: residual add + dynamic-tanh
+// norm (with the embedding lookup as its first form), exact gelu, and the passes that turn a fused projection row
+// into queries and cache rows.  Storage is bf16 or fp32 (template), arithmetic fp32.
+#include <cuda_bf16.h>
+#include <cuda_runtime.h>
+
+#include "host_common.h"
+#include "../../include/l3ci_mixers.h"
+#include "mixer_types.cuh"
+#include "ptx_sm100.cuh"
+#include "warp_reduce.cuh"
+
+namespace l3ci {
+namespace {
+
+// ---- x += y (or x = table[token]);  out = tanh(alpha x) * w + b ------------------------------------------------
+// A CTA per row; VEC elements per access (4: 16 bytes of the fp32 stream, 8 or 16 of the storage type).
+template <typename S, int VEC>
+__global__ void __launch_bounds__(512)
+add_dyn_tanh_kernel(const S* __restrict__ y, const long long* __restrict__ tokens, const S* __restrict__ table, long long vocab,
+                    float* __restrict__ x, const float* __restrict__ w, const float* __restrict__ b, float alpha,
+                    S* __restrict__ out, int width) {
+  pdl_wait();
+  pdl_launch_dependents();
+  const long long row = blockIdx.x;
+  float* xr = x + row * width;
+  const S* add = y ? y + row * width : nullptr;
+  if (tokens) {
+    const long long tok = tokens[row];
+    add = tok >= 0 && tok < vocab ? table + tok * width : nullptr;
+  }
+  for (int c = threadIdx.x * VEC; c < width; c += blockDim.x * VEC) {
+    float v[VEC], a[VEC];
+    if (tokens) {
+#pragma unroll
+      for (int i = 0; i < VEC; ++i) v[i] = 0.f;
+    } else {
+      load_vec<float, VEC>(xr + c, v);
+    }
+    if (add) {
+      load_vec<S, VEC>(add + c, a);
+#pragma unroll
+      for (int i = 0; i < VEC; ++i) v[i] += a[i];
+    }
+    if (add || tokens) store_vec<float, VEC>(xr + c, v);
+    float wv[VEC], bv[VEC];
+    load_vec<float, VEC>(w + c, wv);
+    load_vec<float, VEC>(b + c, bv);
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) v[i] = fmaf(tanhf(alpha * v[i]), wv[i], bv[i]);
+    store_vec<S, VEC>(out + row * width + c, v);
+  }
+}
+
+template <typename S, int VEC>
+__global__ void __launch_bounds__(256) gelu_kernel(const S* __restrict__ z, S* __restrict__ out, long long n) {
+  pdl_wait();
+  pdl_launch_dependents();
+  const long long i0 = ((long long)blockIdx.x * 256 + threadIdx.x) * VEC;
+  if (i0 >= n) return;
+  float v[VEC];
+  load_vec<S, VEC>(z + i0, v);
+#pragma unroll
+  for (int i = 0; i < VEC; ++i) v[i] = 0.5f * v[i] * (1.f + erff(v[i] * 0.70710678118654752f));
+  store_vec<S, VEC>(out + i0, v);
+}
+
+// ---- latent attention: query rotation in place, latent norm, key rotation, cache row ---------------------------
+struct LatentRow {
+  long long qd_stride, table_rows, cache_sb, cache_st, cache_len;
+  int T, H, dim, rot, rank;
+  float eps;
+};
+
+template <typename S>
+__global__ void __launch_bounds__(256)
+latent_cache_kernel(S* __restrict__ qd, const float* __restrict__ table, const float* __restrict__ nw, S* __restrict__ cache,
+                    const int* __restrict__ positions, const LatentRow p) {
+  __shared__ float red[32];
+  pdl_wait();
+  pdl_launch_dependents();
+  const long long row = blockIdx.x;
+  const int b = (int)(row / p.T), t = (int)(row % p.T);
+  const long long pos = (long long)positions[b] + t;
+  if (pos < 0 || pos >= p.table_rows || pos >= p.cache_len) return;
+  S* r = qd + row * p.qd_stride;
+  const int half = p.rot / 2, head = p.dim + p.rot;
+  const float* cs = table + pos * p.rot;
+  const S* down = r + (long long)p.H * head;
+  S* dst = cache + b * p.cache_sb + pos * p.cache_st;
+  float ss = 0.f;
+  for (int c = threadIdx.x; c < p.rank; c += blockDim.x) {
+    const float v = to_f32(down[c]);
+    ss = fmaf(v, v, ss);
+  }
+  ss = cta_sum(ss, red, blockDim.x / kWarp);
+  const float inv = __frsqrt_rn(__fadd_rn(__fdiv_rn(ss, (float)p.rank), p.eps));
+  for (int c = threadIdx.x; c < p.rank; c += blockDim.x) dst[c] = from_f32<S>(to_f32(down[c]) * inv * nw[c]);
+  // the shared key part, then the query heads: (H + 1) * rot/2 pairs
+  for (int i = threadIdx.x; i < (p.H + 1) * half; i += blockDim.x) {
+    const int n = i / half, j = i % half;
+    const float c = cs[2 * j], s = cs[2 * j + 1];
+    const S* src = n < p.H ? r + (long long)n * head + p.dim : down + p.rank;
+    const float u = to_f32(src[j]), v = to_f32(src[j + half]);
+    S* to = n < p.H ? r + (long long)n * head + p.dim : dst + p.rank;
+    to[j] = from_f32<S>(u * c - v * s);
+    to[j + half] = from_f32<S>(v * c + u * s);
+  }
+}
+
+// ---- k and v columns of a projection row into the caches ------------------------------------------------------
+template <typename S, int VEC>
+__global__ void __launch_bounds__(128)
+kv_cache_write_kernel(const S* __restrict__ src, long long stride, long long k_col, int k_width, long long v_col, int v_width,
+                      S* __restrict__ ck, long long k_sb, long long k_st, S* __restrict__ cv, long long v_sb, long long v_st,
+                      long long cache_len, const int* __restrict__ positions, int T) {
+  pdl_wait();
+  pdl_launch_dependents();
+  const long long row = blockIdx.x;
+  const int b = (int)(row / T), t = (int)(row % T);
+  const long long pos = (long long)positions[b] + t;
+  if (pos < 0 || pos >= cache_len) return;
+  const S* r = src + row * stride;
+  for (int i = threadIdx.x * VEC; i < k_width + v_width; i += blockDim.x * VEC) {
+    const bool is_k = i < k_width;
+    const S* from = is_k ? r + k_col + i : r + v_col + (i - k_width);
+    S* to = is_k ? ck + b * k_sb + pos * k_st + i : cv + b * v_sb + pos * v_st + (i - k_width);
+    copy_vec<S, VEC>(from, to);
+  }
+}
+
+bool bad_dtype(int dtype) { return dtype != L3CI_BF16 && dtype != L3CI_F32; }
+template <typename S>
+bool vec_ok(const void* p, int vec) { return (reinterpret_cast<uintptr_t>(p) % (vec * sizeof(S))) == 0; }
+
+template <typename S>
+int add_dyn_tanh_typed(const void* y, const int64_t* tokens, const void* table, int64_t vocab, float* x, const float* w,
+                       const float* b, float alpha, void* out, int64_t rows, int64_t width, cudaStream_t stream) {
+  const bool v4 = width % 4 == 0 && vec_ok<S>(y, 4) && vec_ok<S>(table, 4) && vec_ok<S>(out, 4) && vec_ok<float>(x, 4) &&
+                  vec_ok<float>(w, 4) && vec_ok<float>(b, 4);
+  const int units = (int)(v4 ? width / 4 : width);
+  int threads = 32;
+  while (threads < 512 && threads < units) threads *= 2;
+  auto go = [&](auto kernel) -> int {
+    L3CI_LAUNCH("add_dyn_tanh_kernel", kernel, dim3((unsigned)rows), dim3(threads), 0, stream, static_cast<const S*>(y),
+                reinterpret_cast<const long long*>(tokens), static_cast<const S*>(table), (long long)vocab, x, w, b, alpha,
+                static_cast<S*>(out), (int)width);
+    return L3CI_OK;
+  };
+  return v4 ? go(add_dyn_tanh_kernel<S, 4>) : go(add_dyn_tanh_kernel<S, 1>);
+}
+
+template <typename S>
+int gelu_typed(const void* z, void* out, int64_t n, cudaStream_t stream) {
+  constexpr int kVec = 16 / sizeof(S);
+  const bool v = n % kVec == 0 && vec_ok<S>(z, kVec) && vec_ok<S>(out, kVec);
+  const long long units = v ? n / kVec : n, ctas = (units + 255) / 256;
+  if (ctas > 0x7fffffffLL) return fail(L3CI_ERR_INVALID, "gelu: tensor too large");
+  auto go = [&](auto kernel) -> int {
+    L3CI_LAUNCH("gelu_kernel", kernel, dim3((unsigned)ctas), dim3(256), 0, stream, static_cast<const S*>(z), static_cast<S*>(out), (long long)n);
+    return L3CI_OK;
+  };
+  return v ? go(gelu_kernel<S, kVec>) : go(gelu_kernel<S, 1>);
+}
+
+}  // namespace
+}  // namespace l3ci
+
+extern "C" {
+
+const char* l3ci_mixers_last_error(void) { return l3ci_last_error(); }
+int l3ci_mixers_set_programmatic_launch(int on) { return l3ci_set_programmatic_launch(on); }
+
+int l3ci_add_dyn_tanh(const void* y, const int64_t* tokens, const void* table, int64_t vocab, float* x, const float* weight,
+                      const float* bias, float alpha, void* out, int64_t rows, int64_t width, int32_t dtype,
+                      l3ci_stream_t stream_) {
+  using namespace l3ci;
+  clear_error();
+  if (rows < 0 || width <= 0 || width > 0x7fffffffLL || rows > 0x7fffffffLL || bad_dtype(dtype))
+    return fail(L3CI_ERR_INVALID, "add_dyn_tanh: rows=%lld width=%lld dtype=%d", (long long)rows, (long long)width, dtype);
+  if (rows == 0) return L3CI_OK;
+  if (!x || !weight || !bias || !out || (tokens && (!table || vocab <= 0 || y)))
+    return fail(L3CI_ERR_INVALID, "add_dyn_tanh: null pointer, or both y and tokens");
+  cudaStream_t s = reinterpret_cast<cudaStream_t>(stream_);
+  return dtype == L3CI_BF16 ? add_dyn_tanh_typed<__nv_bfloat16>(y, tokens, table, vocab, x, weight, bias, alpha, out, rows, width, s)
+                            : add_dyn_tanh_typed<float>(y, tokens, table, vocab, x, weight, bias, alpha, out, rows, width, s);
+}
+
+int l3ci_gelu(const void* z, void* out, int64_t n, int32_t dtype, l3ci_stream_t stream_) {
+  using namespace l3ci;
+  clear_error();
+  if (n < 0 || bad_dtype(dtype)) return fail(L3CI_ERR_INVALID, "gelu: n=%lld dtype=%d", (long long)n, dtype);
+  if (n == 0) return L3CI_OK;
+  if (!z || !out) return fail(L3CI_ERR_INVALID, "gelu: null pointer");
+  cudaStream_t s = reinterpret_cast<cudaStream_t>(stream_);
+  return dtype == L3CI_BF16 ? gelu_typed<__nv_bfloat16>(z, out, n, s) : gelu_typed<float>(z, out, n, s);
+}
+
+int l3ci_latent_cache(void* qd, int64_t qd_stride, const float* table, int64_t table_rows, const float* norm_weight, float eps,
+                      void* cache, int64_t cache_sb, int64_t cache_st, int64_t cache_len, const int32_t* positions, int32_t B,
+                      int32_t T, int32_t H, int32_t dim, int32_t rot_dim, int32_t rank, int32_t dtype, l3ci_stream_t stream_) {
+  using namespace l3ci;
+  clear_error();
+  if (B < 0 || T < 0 || H <= 0 || dim < 0 || rot_dim < 0 || rot_dim % 2 || rank <= 0 || bad_dtype(dtype) ||
+      qd_stride < (int64_t)H * (dim + rot_dim) + rank + rot_dim || cache_st < rank + rot_dim)
+    return fail(L3CI_ERR_INVALID, "latent_cache: B=%d T=%d H=%d dim=%d rot_dim=%d rank=%d", B, T, H, dim, rot_dim, rank);
+  if (B == 0 || T == 0) return L3CI_OK;
+  if (!qd || (!table && rot_dim) || !norm_weight || !cache || !positions) return fail(L3CI_ERR_INVALID, "latent_cache: null pointer");
+  const long long rows = (long long)B * T;
+  if (rows > 0x7fffffffLL) return fail(L3CI_ERR_INVALID, "latent_cache: too many rows");
+  LatentRow p{qd_stride, table_rows, cache_sb, cache_st, cache_len, T, H, dim, rot_dim, rank, eps};
+  cudaStream_t s = reinterpret_cast<cudaStream_t>(stream_);
+  if (dtype == L3CI_BF16)
+    L3CI_LAUNCH("latent_cache_kernel", latent_cache_kernel<__nv_bfloat16>, dim3((unsigned)rows), dim3(256), 0, s,
+                static_cast<__nv_bfloat16*>(qd), table, norm_weight, static_cast<__nv_bfloat16*>(cache), positions, p);
+  else
+    L3CI_LAUNCH("latent_cache_kernel", latent_cache_kernel<float>, dim3((unsigned)rows), dim3(256), 0, s, static_cast<float*>(qd),
+                table, norm_weight, static_cast<float*>(cache), positions, p);
+  return L3CI_OK;
+}
+
+int l3ci_kv_cache_write(const void* src, int64_t src_stride, int64_t k_col, int64_t k_width, int64_t v_col, int64_t v_width,
+                        void* cache_k, int64_t k_sb, int64_t k_st, void* cache_v, int64_t v_sb, int64_t v_st, int64_t cache_len,
+                        const int32_t* positions, int32_t B, int32_t T, int32_t dtype, l3ci_stream_t stream_) {
+  using namespace l3ci;
+  clear_error();
+  if (B < 0 || T < 0 || k_width <= 0 || v_width <= 0 || k_width + v_width > 0x7fffffffLL || k_col < 0 || v_col < 0 ||
+      k_col + k_width > src_stride || v_col + v_width > src_stride || bad_dtype(dtype))
+    return fail(L3CI_ERR_INVALID, "kv_cache_write: B=%d T=%d widths %lld %lld", B, T, (long long)k_width, (long long)v_width);
+  if (B == 0 || T == 0) return L3CI_OK;
+  if (!src || !cache_k || !cache_v || !positions) return fail(L3CI_ERR_INVALID, "kv_cache_write: null pointer");
+  const long long rows = (long long)B * T;
+  if (rows > 0x7fffffffLL) return fail(L3CI_ERR_INVALID, "kv_cache_write: too many rows");
+  cudaStream_t s = reinterpret_cast<cudaStream_t>(stream_);
+  auto typed = [&](auto zero) -> int {
+    using S = decltype(zero);
+    constexpr int kVec = 16 / sizeof(S);
+    const int64_t all = src_stride | k_col | k_width | v_col | v_width | k_sb | k_st | v_sb | v_st;
+    const bool v = all % kVec == 0 && aligned16(src) && aligned16(cache_k) && aligned16(cache_v);
+    auto go = [&](auto kernel) -> int {
+      L3CI_LAUNCH("kv_cache_write_kernel", kernel, dim3((unsigned)rows), dim3(128), 0, s, static_cast<const S*>(src), (long long)src_stride,
+                  (long long)k_col, (int)k_width, (long long)v_col, (int)v_width, static_cast<S*>(cache_k), (long long)k_sb,
+                  (long long)k_st, static_cast<S*>(cache_v), (long long)v_sb, (long long)v_st, (long long)cache_len, positions, T);
+      return L3CI_OK;
+    };
+    return v ? go(kv_cache_write_kernel<S, kVec>) : go(kv_cache_write_kernel<S, 1>);
+  };
+  return dtype == L3CI_BF16 ? typed(__nv_bfloat16{}) : typed(float{});
+}
+
+}  // extern "C"

@@ -1,0 +1,51 @@
+// Storage-type helpers of the mixer kernels: bf16 or fp32 in memory, fp32 in registers.
+#pragma once
+
+#include <cuda_bf16.h>
+#include <stdint.h>
+
+#include "bf16x8.cuh"
+
+namespace l3ci {
+
+__device__ __forceinline__ float to_f32(float v) { return v; }
+__device__ __forceinline__ float to_f32(__nv_bfloat16 v) { return __bfloat162float(v); }
+template <typename S>
+__device__ __forceinline__ S from_f32(float v);
+template <>
+__device__ __forceinline__ float from_f32<float>(float v) { return v; }
+template <>
+__device__ __forceinline__ __nv_bfloat16 from_f32<__nv_bfloat16>(float v) { return __float2bfloat16_rn(v); }
+
+template <int BYTES>
+struct Raw;
+template <>
+struct Raw<2> { using type = uint16_t; };
+template <>
+struct Raw<4> { using type = uint32_t; };
+template <>
+struct Raw<8> { using type = uint2; };
+template <>
+struct Raw<16> { using type = uint4; };
+
+template <typename S, int VEC>
+__device__ __forceinline__ void load_vec(const S* p, float (&f)[VEC]) {
+  union { typename Raw<VEC * sizeof(S)>::type raw; S s[VEC]; } u;
+  u.raw = *reinterpret_cast<const typename Raw<VEC * sizeof(S)>::type*>(p);
+#pragma unroll
+  for (int i = 0; i < VEC; ++i) f[i] = to_f32(u.s[i]);
+}
+template <typename S, int VEC>
+__device__ __forceinline__ void store_vec(S* p, const float (&f)[VEC]) {
+  union { typename Raw<VEC * sizeof(S)>::type raw; S s[VEC]; } u;
+#pragma unroll
+  for (int i = 0; i < VEC; ++i) u.s[i] = from_f32<S>(f[i]);
+  *reinterpret_cast<typename Raw<VEC * sizeof(S)>::type*>(p) = u.raw;
+}
+template <typename S, int VEC>
+__device__ __forceinline__ void copy_vec(const S* from, S* to) {
+  using R = typename Raw<VEC * sizeof(S)>::type;
+  *reinterpret_cast<R*>(to) = *reinterpret_cast<const R*>(from);
+}
+
+}  // namespace l3ci

@@ -47,3 +47,11 @@ def precompute_freqs_cis(dim: int, end: int, theta: float = 10000.0, use_scaled:
     t = torch.arange(end, dtype=torch.float32)
     angles = torch.outer(t, freqs)
     return torch.view_as_real(torch.polar(torch.ones_like(angles), angles)).flatten(1)
+
+
+def rotation_table(dims: int, end: int, base: float) -> torch.Tensor:
+    """fp32 [end, dims] table in the layout above for frequencies base^(-2i/dims), without scaling.  Angles are formed
+    in float64 and rounded once, so that far positions are as exact as near ones."""
+    freqs = float(base) ** (-torch.arange(0, dims, 2, dtype=torch.float64) / dims)
+    angles = torch.outer(torch.arange(end, dtype=torch.float64), freqs)
+    return torch.stack([angles.cos(), angles.sin()], dim=-1).flatten(1).float().contiguous()
