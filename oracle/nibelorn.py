@@ -83,6 +83,29 @@ def latent_attention(h, w, m, eps):
     return out.reshape(T, H * V) @ w["o"].to(F64).T
 
 
+def cached_attention(q, k, v, start, scale, cap=0.0, temp=None):
+    """Softmax attention of q[t, H, D] at positions start + t over k[j, G, D], v[j, G, V]: keys j <= start + t."""
+    T, H, _ = q.shape
+    S, G, _ = k.shape
+    pos = torch.arange(start, start + T)
+    factor = query_temperature(pos, *temp) if temp else torch.ones(T, dtype=F64)
+    hidden = torch.arange(S)[None, :] > pos[:, None]
+    out = torch.empty(T, H, v.shape[-1], dtype=F64)
+    for n in range(H):
+        g = n // (H // G)
+        s = (q[:, n].to(F64) * factor[:, None]) @ k[:, g].to(F64).T * scale
+        if cap:
+            s = softcap(s, cap)
+        out[:, n] = torch.softmax(s.masked_fill(hidden, -math.inf), dim=-1) @ v[:, g].to(F64)
+    return out
+
+
+def differential_combine(a1, a2, lam, diff, eps, gate=None):
+    """a1, a2 [t, H, V]: the maps' outputs; gate [t, H] before the sigmoid."""
+    o = rms(a1 - lam * a2, eps) * (1.0 - diff)
+    return o if gate is None else o * torch.sigmoid(gate.to(F64))[..., None]
+
+
 def differential_lambda(w, diff):
     def dot(a, b):
         return (w[a].to(F64) * w[b].to(F64)).sum()
