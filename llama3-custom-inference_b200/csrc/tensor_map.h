@@ -47,4 +47,22 @@ inline int make_kv_map(CUtensorMap* map, const void* base, int D, int n_seq, int
 }
 
 
+// Rank-4 map over a [B, G, n_rows, width] view whose rows are cut into 64-column boxes of `tile` rows of one head;
+// columns and rows beyond the view read as 0.  width and the strides: multiples of 8.
+inline int make_rows_map(CUtensorMap* map, const void* base, int width, int n_rows, int G, int B, long long st, long long sh,
+                         long long sb, int tile) {
+  auto enc = tensor_map_encoder();
+  if (!enc) return fail(L3CI_ERR_CUDA, "cuTensorMapEncodeTiled is not available");
+  const cuuint64_t any = ((cuuint64_t)width * 2 + 15) / 16 * 16;   // a dimension of extent 1 may carry any stride
+  cuuint64_t dims[4] = {(cuuint64_t)width, (cuuint64_t)n_rows, (cuuint64_t)G, (cuuint64_t)B};
+  cuuint64_t strides[3] = {n_rows > 1 ? (cuuint64_t)st * 2 : any, G > 1 ? (cuuint64_t)sh * 2 : any, B > 1 ? (cuuint64_t)sb * 2 : any};
+  cuuint32_t box[4] = {64u, (cuuint32_t)tile, 1u, 1u};
+  cuuint32_t estr[4] = {1u, 1u, 1u, 1u};
+  const CUresult r = enc(map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 4, const_cast<void*>(base), dims, strides, box, estr,
+                         CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
+                         CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
+  if (r != CUDA_SUCCESS) return fail(L3CI_ERR_CUDA, "cuTensorMapEncodeTiled failed with %d", (int)r);
+  return L3CI_OK;
+}
+
 }  // namespace l3ci
