@@ -34,9 +34,9 @@ class AttnArgs(C.Structure):
 
 
 def tc_sizes_ok(Da: int, Db: int, Dv: int) -> bool:
-    """Sizes the tcgen05 kernel of `attention` takes (variant TC): parts that fit its shared-memory tiles, rows of whole
-    16-byte vectors."""
-    return False
+    """Sizes the tcgen05 kernel of `attention` takes for one map (variant TC): parts that fit its shared-memory tiles, rows of
+    whole 16-byte vectors."""
+    return 0 < Da <= 128 and Db <= 64 and Dv <= 128 and Da % 8 == 0 and Db % 8 == 0 and Dv % 8 == 0
 
 
 _lib = None

@@ -198,6 +198,73 @@ def test_differential_attention_finds_a_single_key(pkg, device, m, key):
                                                                         boost=(m, key), variant=v))
 
 
+@pytest.mark.parametrize("H,G,D,V", [(4, 1, 32, 64), (6, 2, 24, 40), (3, 3, 64, 128), (16, 4, 64, 128), (2, 1, 8, 8)])
+@pytest.mark.parametrize("T,start", [(128, 0), (129, 0), (300, 0), (130, 77), (128, 128), (5, 260)])
+def test_differential_attention_of_a_prompt(pkg, device, H, G, D, V, T, start):
+    """The tcgen05 kernel: whole prompts and later portions, more items than SMs and fewer."""
+    for cap in (0.0, 20.0):
+        run_variants(pkg, device, BF16, (3,), lambda v: differential_case(pkg, device, BF16, 2, T, H, G, D, V, (start, start),
+                                                                          start + T + 10, cap=cap, variant=v))
+
+
+def test_differential_attention_of_a_long_prompt(pkg, device):
+    run_variants(pkg, device, BF16, (3,), lambda v: differential_case(pkg, device, BF16, 1, 1500, 16, 4, 32, 64, (0,), 1500, variant=v))
+
+
+@pytest.mark.parametrize("cap", [0.0, 1.0, 6.0])
+@pytest.mark.parametrize("temp", [(0.0, 0.0), (1.5, 7.0), (-0.9, 3.0)])
+def test_prompt_scores_beyond_the_cap(pkg, device, cap, temp):
+    """Scores far outside the cap's near-linear range; temperatures that grow, and that turn negative."""
+    run_variants(pkg, device, BF16, (2, 3), lambda v: differential_case(pkg, device, BF16, 1, 200, 4, 2, 32, 64, (40,), 240, cap=cap,
+                                                                        temp=temp, variant=v, q_scale=2.0))
+
+
+@pytest.mark.parametrize("m", [0, 1])
+@pytest.mark.parametrize("key", [0, 1, 127, 128, 255, 256, 700])
+def test_prompt_differential_attention_finds_a_single_key(pkg, device, m, key):
+    def make(v):
+        B, T, start, H, G, D, V = 1, 140, 700, 2, 1, 32, 64
+        q, k, val = rand(B, T, H, 2 * D, seed=1), rand(B, 840, G, 2 * D, seed=2), rand(B, 840, G, V, seed=3)
+        k[0, key, 0, m * D:(m + 1) * D] = (40.0 * q[0, 139, 1, m * D:(m + 1) * D].double() / q[0, 139, 1, m * D:(m + 1) * D].double().norm()).to(BF16)
+        out = torch.empty(B, T, H, V, dtype=BF16, device=device)
+        pkg.mixers.attention(q.to(device), k.to(device), val.to(device), out, torch.full((1,), start, dtype=torch.int32, device=device),
+                             maps=2, scale=0.2, softcap=30.0, lambda_=0.4, post=0.6, eps=1e-5, start_pos=start, variant=v)
+        a = [ref.cached_attention(q[0, ..., i * D:(i + 1) * D], k[0, ..., i * D:(i + 1) * D], val[0], start, 0.2, 30.0) for i in range(2)]
+        return out[0], ref.differential_combine(a[0], a[1], 0.4, 0.4, 1e-5)
+
+    run_variants(pkg, device, BF16, (1, 2, 3), make)
+
+
+@pytest.mark.parametrize("H,D,R,V", [(3, 64, 16, 48), (5, 128, 64, 128), (2, 24, 8, 40), (4, 72, 64, 64), (1, 128, 32, 72), (7, 64, 64, 128)])
+@pytest.mark.parametrize("T,start", [(128, 0), (257, 0), (700, 0), (130, 77), (128, 128), (40, 260)])
+def test_expanded_latent_attention_of_a_prompt(pkg, device, H, D, R, V, T, start):
+    """Keys and values per head, the rotated key part shared by the heads and lying in other rows than the rest."""
+    B, S, scale = 2, start + T, 1.4 / math.sqrt(D + R)
+    q, kv, rows = rand(B, T, H, D + R, seed=1), rand(B, S, H * (D + V), seed=2), rand(B, S + 5, 16 + R, seed=3)
+    out = torch.empty(B, T, H, V, dtype=BF16, device=device)
+    dq, dkv, drows = q.to(device), kv.to(device), rows.to(device)
+    positions = torch.full((B,), start, dtype=torch.int32, device=device)
+    for variant in (1, 3):
+        out.zero_()
+        pkg.mixers.attention(dq[..., :D], dkv[..., :H * D].view(B, S, H, D), dkv[..., H * D:].view(B, S, H, V), out, positions,
+                             qb=dq[..., D:], kb=drows[:, :S, None, 16:].expand(B, S, H, R), scale=scale, start_pos=start,
+                             variant=variant)
+        torch.cuda.synchronize()
+        for b in range(B):
+            k = torch.cat([kv[b, :, :H * D].view(S, H, D), rows[b, :S, None, 16:].expand(S, H, R)], dim=-1)
+            close(out[b], ref.cached_attention(q[b], k, kv[b, :, H * D:].view(S, H, V), start, scale), BF16, f"variant {variant}")
+
+
+def test_one_map_without_a_second_part(pkg, device):
+    B, T, S, H, G, D, V = 1, 200, 230, 6, 2, 96, 56
+    q, k, v = rand(B, T, H, D, seed=1), rand(B, S, G, D, seed=2), rand(B, S, G, V, seed=3)
+    for variant in (1, 2, 3):
+        out = torch.empty(B, T, H, V, dtype=BF16, device=device)
+        pkg.mixers.attention(q.to(device), k.to(device), v.to(device), out, torch.full((1,), 30, dtype=torch.int32, device=device),
+                             scale=0.15, start_pos=30, variant=variant)
+        close(out[0], ref.cached_attention(q[0], k[0], v[0], 30, 0.15), BF16, f"variant {variant}")
+
+
 def test_attention_reads_nothing_beyond_the_position(pkg, device):
     """What lies in the cache after a query's position (an earlier holder's rows, even NaN) does not enter."""
     B, T, H, C, R, L = 1, 1, 4, 64, 16, 512
