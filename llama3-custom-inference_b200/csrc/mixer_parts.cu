@@ -108,25 +108,108 @@ latent_cache_kernel(S* __restrict__ qd, const float* __restrict__ table, const f
   }
 }
 
+// The same in 16-byte vectors (bf16; rank a multiple of 8, rot_dim of 16, rows on 16 bytes): all loads of a row are in
+// flight before the reduction of its latent.
+constexpr int kLatentThreads = 128;
+constexpr int kLatentVecs = 8;   // latent vectors per thread at most: rank <= 8192
+
+template <int VPT>
+__global__ void __launch_bounds__(kLatentThreads)
+latent_cache_vec_kernel(__nv_bfloat16* __restrict__ qd, const float* __restrict__ table, const float* __restrict__ nw,
+                        __nv_bfloat16* __restrict__ cache, const int* __restrict__ positions, const LatentRow p) {
+  __shared__ float red[32];
+  pdl_wait();
+  pdl_launch_dependents();
+  const long long row = blockIdx.x;
+  const int b = (int)(row / p.T), t = (int)(row % p.T), tid = threadIdx.x;
+  const long long pos = (long long)positions[b] + t;
+  if (pos < 0 || pos >= p.table_rows || pos >= p.cache_len) return;
+  __nv_bfloat16* r = qd + row * p.qd_stride;
+  const int head = p.dim + p.rot, half = p.rot / 2, per_head = half / 8;   // vector pairs per head
+  const __nv_bfloat16* down = r + (long long)p.H * head;
+  __nv_bfloat16* dst = cache + b * p.cache_sb + pos * p.cache_st;
+  const float* cs = table + pos * p.rot;
+  uint4 c[VPT];
+#pragma unroll
+  for (int i = 0; i < VPT; ++i) {
+    const int v = tid + i * kLatentThreads;
+    c[i] = v * 8 < p.rank ? *reinterpret_cast<const uint4*>(down + v * 8) : make_uint4(0, 0, 0, 0);
+  }
+  for (int i = tid; i < (p.H + 1) * per_head; i += kLatentThreads) {
+    const int n = i / per_head, j = (i - n * per_head) * 8;
+    const __nv_bfloat16* src = n < p.H ? r + (long long)n * head + p.dim : down + p.rank;
+    __nv_bfloat16* to = n < p.H ? r + (long long)n * head + p.dim : dst + p.rank;
+    const uint4 uv = *reinterpret_cast<const uint4*>(src + j), vv = *reinterpret_cast<const uint4*>(src + j + half);
+    float u[8], v[8], x[8], y[8];
+    unpack8(uv, u);
+    unpack8(vv, v);
+#pragma unroll
+    for (int k = 0; k < 8; k += 2) {
+      const float4 f = __ldg(reinterpret_cast<const float4*>(cs + 2 * (j + k)));   // cos, sin of pairs j + k, j + k + 1
+      x[k] = u[k] * f.x - v[k] * f.y;
+      y[k] = v[k] * f.x + u[k] * f.y;
+      x[k + 1] = u[k + 1] * f.z - v[k + 1] * f.w;
+      y[k + 1] = v[k + 1] * f.z + u[k + 1] * f.w;
+    }
+    *reinterpret_cast<uint4*>(to + j) = pack8(x);
+    *reinterpret_cast<uint4*>(to + j + half) = pack8(y);
+  }
+  float ss = 0.f;
+#pragma unroll
+  for (int i = 0; i < VPT; ++i) {
+    float f[8];
+    unpack8(c[i], f);
+#pragma unroll
+    for (int k = 0; k < 8; ++k) ss = fmaf(f[k], f[k], ss);
+  }
+  ss = cta_sum(ss, red, kLatentThreads / kWarp);
+  const float inv = __frsqrt_rn(__fadd_rn(__fdiv_rn(ss, (float)p.rank), p.eps));
+#pragma unroll
+  for (int i = 0; i < VPT; ++i) {
+    const int v = tid + i * kLatentThreads;
+    if (v * 8 < p.rank) {
+      float f[8];
+      unpack8(c[i], f);
+      const float4 w0 = __ldg(reinterpret_cast<const float4*>(nw + v * 8)), w1 = __ldg(reinterpret_cast<const float4*>(nw + v * 8 + 4));
+      const float w[8] = {w0.x, w0.y, w0.z, w0.w, w1.x, w1.y, w1.z, w1.w};
+#pragma unroll
+      for (int k = 0; k < 8; ++k) f[k] = f[k] * inv * w[k];
+      *reinterpret_cast<uint4*>(dst + v * 8) = pack8(f);
+    }
+  }
+}
+
 // ---- k and v columns of a projection row into the caches ------------------------------------------------------
+// A thread copies kCopies accesses of VEC elements, all loaded before the first is stored.
+constexpr int kCopies = 4;
+
 template <typename S, int VEC>
 __global__ void __launch_bounds__(128)
 kv_cache_write_kernel(const S* __restrict__ src, long long stride, long long k_col, int k_width, long long v_col, int v_width,
                       S* __restrict__ ck, long long k_sb, long long k_st, S* __restrict__ cv, long long v_sb, long long v_st,
-                      long long cache_len, const int* __restrict__ positions, int T) {
+                      long long cache_len, const int* __restrict__ positions, int T, int rows) {
   pdl_wait();
   pdl_launch_dependents();
-  const long long row = blockIdx.x;
-  const int b = (int)(row / T), t = (int)(row % T);
-  const long long pos = (long long)positions[b] + t;
-  if (pos < 0 || pos >= cache_len) return;
-  const S* r = src + row * stride;
-  for (int i = threadIdx.x * VEC; i < k_width + v_width; i += blockDim.x * VEC) {
+  using R = typename Raw<VEC * sizeof(S)>::type;
+  const unsigned per_row = (k_width + v_width) / VEC;
+  R data[kCopies];
+  S* to[kCopies];
+#pragma unroll
+  for (int u = 0; u < kCopies; ++u) {
+    to[u] = nullptr;
+    const long long id = ((long long)blockIdx.x * kCopies + u) * 128 + threadIdx.x;
+    if (id >= (long long)rows * per_row) continue;
+    const long long row = per_row * (long long)rows <= 0xffffffffLL ? (unsigned)id / per_row : id / per_row;
+    const int i = (int)(id - row * per_row) * VEC, b = (int)(row / T), t = (int)(row % T);
+    const long long pos = (long long)positions[b] + t;
+    if (pos < 0 || pos >= cache_len) continue;
     const bool is_k = i < k_width;
-    const S* from = is_k ? r + k_col + i : r + v_col + (i - k_width);
-    S* to = is_k ? ck + b * k_sb + pos * k_st + i : cv + b * v_sb + pos * v_st + (i - k_width);
-    copy_vec<S, VEC>(from, to);
+    data[u] = *reinterpret_cast<const R*>(src + row * stride + (is_k ? k_col + i : v_col + (i - k_width)));
+    to[u] = is_k ? ck + b * k_sb + pos * k_st + i : cv + b * v_sb + pos * v_st + (i - k_width);
   }
+#pragma unroll
+  for (int u = 0; u < kCopies; ++u)
+    if (to[u]) *reinterpret_cast<R*>(to[u]) = data[u];
 }
 
 bool bad_dtype(int dtype) { return dtype != L3CI_BF16 && dtype != L3CI_F32; }
@@ -210,6 +293,17 @@ int l3ci_latent_cache(void* qd, int64_t qd_stride, const float* table, int64_t t
   if (rows > 0x7fffffffLL) return fail(L3CI_ERR_INVALID, "latent_cache: too many rows");
   LatentRow p{qd_stride, table_rows, cache_sb, cache_st, cache_len, T, H, dim, rot_dim, rank, eps};
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream_);
+  const bool vec = dtype == L3CI_BF16 && rank % 8 == 0 && rot_dim % 16 == 0 && dim % 8 == 0 && qd_stride % 8 == 0 && cache_sb % 8 == 0 &&
+                   cache_st % 8 == 0 && rank <= 8 * kLatentVecs * kLatentThreads && aligned16(qd) && aligned16(cache) &&
+                   aligned16(table) && aligned16(norm_weight);
+  if (vec) {
+    auto go = [&](auto kernel) -> int {
+      L3CI_LAUNCH("latent_cache_vec_kernel", kernel, dim3((unsigned)rows), dim3(kLatentThreads), 0, s, static_cast<__nv_bfloat16*>(qd),
+                  table, norm_weight, static_cast<__nv_bfloat16*>(cache), positions, p);
+      return L3CI_OK;
+    };
+    return rank <= 8 * kLatentThreads ? go(latent_cache_vec_kernel<1>) : go(latent_cache_vec_kernel<kLatentVecs>);
+  }
   if (dtype == L3CI_BF16)
     L3CI_LAUNCH("latent_cache_kernel", latent_cache_kernel<__nv_bfloat16>, dim3((unsigned)rows), dim3(256), 0, s,
                 static_cast<__nv_bfloat16*>(qd), table, norm_weight, static_cast<__nv_bfloat16*>(cache), positions, p);
@@ -237,13 +331,15 @@ int l3ci_kv_cache_write(const void* src, int64_t src_stride, int64_t k_col, int6
     constexpr int kVec = 16 / sizeof(S);
     const int64_t all = src_stride | k_col | k_width | v_col | v_width | k_sb | k_st | v_sb | v_st;
     const bool v = all % kVec == 0 && aligned16(src) && aligned16(cache_k) && aligned16(cache_v);
-    auto go = [&](auto kernel) -> int {
-      L3CI_LAUNCH("kv_cache_write_kernel", kernel, dim3((unsigned)rows), dim3(128), 0, s, static_cast<const S*>(src), (long long)src_stride,
+    auto go = [&](auto kernel, int width) -> int {
+      const long long units = rows * ((k_width + v_width) / width), per_cta = 128LL * kCopies;
+      if ((units + per_cta - 1) / per_cta > 0x7fffffffLL) return fail(L3CI_ERR_INVALID, "kv_cache_write: too much");
+      L3CI_LAUNCH("kv_cache_write_kernel", kernel, dim3((unsigned)((units + per_cta - 1) / per_cta)), dim3(128), 0, s, static_cast<const S*>(src), (long long)src_stride,
                   (long long)k_col, (int)k_width, (long long)v_col, (int)v_width, static_cast<S*>(cache_k), (long long)k_sb,
-                  (long long)k_st, static_cast<S*>(cache_v), (long long)v_sb, (long long)v_st, (long long)cache_len, positions, T);
+                  (long long)k_st, static_cast<S*>(cache_v), (long long)v_sb, (long long)v_st, (long long)cache_len, positions, T, (int)rows);
       return L3CI_OK;
     };
-    return v ? go(kv_cache_write_kernel<S, kVec>) : go(kv_cache_write_kernel<S, 1>);
+    return v ? go(kv_cache_write_kernel<S, kVec>, kVec) : go(kv_cache_write_kernel<S, 1>, 1);
   };
   return dtype == L3CI_BF16 ? typed(__nv_bfloat16{}) : typed(float{});
 }

@@ -42,10 +42,5 @@ __device__ __forceinline__ void store_vec(S* p, const float (&f)[VEC]) {
   for (int i = 0; i < VEC; ++i) u.s[i] = from_f32<S>(f[i]);
   *reinterpret_cast<typename Raw<VEC * sizeof(S)>::type*>(p) = u.raw;
 }
-template <typename S, int VEC>
-__device__ __forceinline__ void copy_vec(const S* from, S* to) {
-  using R = typename Raw<VEC * sizeof(S)>::type;
-  *reinterpret_cast<R*>(to) = *reinterpret_cast<const R*>(from);
-}
 
 }  // namespace l3ci

@@ -135,13 +135,13 @@ def latent_case(pkg, device, dtype, B, T, H, C, R, starts, L, seed=0, variant=0,
     return out, want
 
 
-@pytest.mark.parametrize("H,C,R", [(1, 16, 8), (5, 40, 24), (8, 128, 16), (16, 512, 64), (20, 96, 32), (3, 200, 8)])
+@pytest.mark.parametrize("H,C,R", [(1, 16, 8), (5, 40, 24), (10, 112, 24), (16, 512, 64), (20, 96, 32), (3, 200, 8)])
 @pytest.mark.parametrize("T,starts", [(1, (0, 70)), (1, (63, 64)), (1, (127, 300)), (2, (62, 62)), (7, (0, 0)), (67, (129, 129))])
 def test_latent_attention_over_the_cache(pkg, device, H, C, R, T, starts):
     run_variants(pkg, device, BF16, (1, 2), lambda v: latent_case(pkg, device, BF16, 2, T, H, C, R, starts, 384, variant=v))
 
 
-@pytest.mark.parametrize("C,R,starts", [(33, 6, (0, 200)), (128, 16, (130, 129))])
+@pytest.mark.parametrize("C,R,starts", [(33, 6, (0, 200)), (112, 24, (130, 129))])
 def test_latent_attention_fp32(pkg, device, C, R, starts):
     run_variants(pkg, device, F32, (0, 1), lambda v: latent_case(pkg, device, F32, 2, 1, 3, C, R, starts, 256, variant=v))
 
@@ -176,7 +176,7 @@ def differential_case(pkg, device, dtype, B, T, H, G, D, V, starts, L, cap=20.0,
     return out, torch.stack(want)
 
 
-@pytest.mark.parametrize("H,G,D,V", [(4, 1, 32, 64), (6, 2, 24, 40), (8, 8, 64, 128), (16, 4, 64, 128), (12, 1, 16, 8), (5, 5, 128, 256)])
+@pytest.mark.parametrize("H,G,D,V", [(4, 1, 40, 56), (6, 2, 24, 40), (8, 8, 64, 128), (16, 4, 64, 128), (12, 1, 16, 8), (5, 5, 128, 256)])
 @pytest.mark.parametrize("T,starts", [(1, (0, 90)), (1, (63, 64)), (2, (126, 126)), (9, (0, 0)), (67, (100, 100))])
 def test_differential_attention_over_the_cache(pkg, device, H, G, D, V, T, starts):
     run_variants(pkg, device, BF16, (1, 2), lambda v: differential_case(pkg, device, BF16, 2, T, H, G, D, V, starts, 320, variant=v))
@@ -198,7 +198,7 @@ def test_differential_attention_finds_a_single_key(pkg, device, m, key):
                                                                         boost=(m, key), variant=v))
 
 
-@pytest.mark.parametrize("H,G,D,V", [(4, 1, 32, 64), (6, 2, 24, 40), (3, 3, 64, 128), (16, 4, 64, 128), (2, 1, 8, 8)])
+@pytest.mark.parametrize("H,G,D,V", [(4, 1, 40, 56), (6, 2, 24, 40), (3, 3, 64, 128), (16, 4, 64, 128), (2, 1, 8, 8)])
 @pytest.mark.parametrize("T,start", [(128, 0), (129, 0), (300, 0), (130, 77), (128, 128), (5, 260)])
 def test_differential_attention_of_a_prompt(pkg, device, H, G, D, V, T, start):
     """The tcgen05 kernel: whole prompts and later portions, more items than SMs and fewer."""
@@ -235,7 +235,7 @@ def test_prompt_differential_attention_finds_a_single_key(pkg, device, m, key):
     run_variants(pkg, device, BF16, (1, 2, 3), make)
 
 
-@pytest.mark.parametrize("H,D,R,V", [(3, 64, 16, 48), (5, 128, 64, 128), (2, 24, 8, 40), (4, 72, 64, 64), (1, 128, 32, 72), (7, 64, 64, 128)])
+@pytest.mark.parametrize("H,D,R,V", [(3, 64, 24, 56), (5, 128, 64, 128), (2, 24, 8, 40), (4, 72, 64, 64), (1, 128, 32, 72), (7, 64, 64, 128)])
 @pytest.mark.parametrize("T,start", [(128, 0), (257, 0), (700, 0), (130, 77), (128, 128), (40, 260)])
 def test_expanded_latent_attention_of_a_prompt(pkg, device, H, D, R, V, T, start):
     """Keys and values per head, the rotated key part shared by the heads and lying in other rows than the rest."""
