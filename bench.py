@@ -1,7 +1,7 @@
 #!/usr/bin/env python
 """Benchmark of the decode hot path on B200.
 
-    python bench.py [--gpus N] [--steps K] [--warmup W] [--workload c2|c1|c3|rmsnorm|rope|c5|prefill]
+    python bench.py [--gpus N] [--steps K] [--warmup W] [--workload c2|c1|c3|rmsnorm|rope|c5|prefill|nibelorn]
                     [--impl ours|reference]
 
 One "step" is one pass of the hot path over one batch of synthetic input: for the default workload (C2) one
@@ -28,6 +28,9 @@ Printed JSON line (rank 0):
   c1, c4_rmsnorm, c4_rope, c5
                  (default workload, N = 1) the other configurations, each with its own roofline; prefill_d64 and
                  prefill_d128: causal prefill attention (the step before the path) against torch's SDPA
+  --workload nibelorn
+                 the Nibelorn decoder at the layer sizes of a 1B model beside the Llama-3 decoder of equal size: prefill and
+                 decode tokens/s at a few batches, and every mixer kernel's roofline beside its Llama-3 counterpart's
   comparators    torch's SDPA on the same GPU tensors; and, at N = 1, the reference's own CUDA kernels rebuilt
                  for sm_100 (oracle/_ref, when present), timed beside this library's calls
 
@@ -265,7 +268,7 @@ def main():
     ap.add_argument("--gpus", type=int, default=1)
     ap.add_argument("--steps", type=int, default=2000)
     ap.add_argument("--warmup", type=int, default=100)
-    ap.add_argument("--workload", default=None, choices=["c1", "c2", "c3", "rmsnorm", "rope", "c5", "prefill"],
+    ap.add_argument("--workload", default=None, choices=["c1", "c2", "c3", "rmsnorm", "rope", "c5", "prefill", "nibelorn"],
                     help="default: c2 as the headline plus the sub-records of the other configurations")
     ap.add_argument("--gen-len", type=int, default=2048, help="c5: tokens generated per sequence")
     ap.add_argument("--batch", type=int, default=64, help="c5: sequences per GPU")
@@ -313,6 +316,8 @@ def main():
 
     if args.workload == "c5":
         line = bench_end_to_end(args, ext, pkg, dev, rank, world)
+    elif args.workload == "nibelorn":
+        line = bench_nibelorn(args, ext, pkg, dev, rank, world)
     elif args.workload == "prefill":
         line = bench_prefill(args, ext, pkg, dev, rank, world)
     elif args.workload in ("rmsnorm", "rope"):
@@ -1035,6 +1040,217 @@ def bench_end_to_end(args, ext, pkg, dev, rank, world):
         except Exception as exc:
             line["comparators"]["sampling_step"] = {"error": str(exc)[:300]}
     return line
+
+
+def bench_nibelorn(args, ext, pkg, dev, rank, world):
+    """The Nibelorn decoder (random weights) at a 1B model's layer sizes: width 2048, 16 layers, latent and differential
+    attention in turn, feed-forward 8192, vocabulary 128256, beside the Llama-3 decoder of the same width, depth,
+    feed-forward size and vocabulary.  Value: decode tokens/s at batch 64 behind 1024-token prompts, by CUDA events
+    around the replayed decode steps of a generation (prefill and graph capture are not in it; prefill is timed alone)."""
+    nb, dl = pkg.nibelorn, pkg.decode_loop
+    latent = nb.LatentAttention(heads=16, dim=128, rot_dim=64, vdim=128, kv_rank=512, scale=192 ** -0.5, rot_base=10000.0)
+    differential = nb.DifferentialAttention(heads=16, kv_heads=4, dim=64, vdim=128, scale=0.125, diff=0.5, softcap=50.0, temp_coef=0.3,
+                                            temp_every=256.0)
+    cfg = nb.NibelornConfig(128256, 2048, 1e-5, tuple(nb.Layer((latent, differential)[i % 2], 8192, i) for i in range(16)))
+    llama = dl.DecoderConfig()
+    short, long = 17, 129
+    shapes = ((64, 1024), (8, 4096), (1, 8192))
+    makers = {
+        "nibelorn": lambda B, L: nb.NibelornDecoder(ext, cfg, dev, B, L, weights=nb.init_weights(cfg, 42 + rank, dev)),
+        "llama3": lambda B, L: dl.Llama3Decoder(ext, llama, dev, B, L, seed=42 + rank),
+    }
+
+    def timed(fn, repeats=3):
+        times = []
+        for _ in range(repeats):
+            sync_all(world)
+            start, end = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+            start.record()
+            fn()
+            end.record()
+            torch.cuda.synchronize()
+            times.append(start.elapsed_time(end))
+        return max_over_ranks(sorted(times)[repeats // 2], world, dev)
+
+    sampler = ClockSampler(dev.index or 0)
+    sampler.start()
+    models, e2e = {}, None
+    for name, make in makers.items():
+        model = make(64, max(64 * (1024 + long), 8 * (4096 + long), 8192 + long) // 64 + 1)
+        models[name] = {}
+        for B, P in shapes:
+            # the same weights behind a cache of this shape: slots and length follow the batch
+            model.cache = pkg.kv_cache.StaticCache([{n: tuple(t.shape[2:]) for n, t in layer.items()} for layer in model.cache.layers],
+                                                   B, P + long, model.dtype, dev)
+            model.max_batch, model.max_len = B, P + long
+            if name == "nibelorn":
+                model._tables = {k: pkg.rope_table.rotation_table(k[0], P + long, k[1]).to(dev) for k in model._tables}
+            else:
+                model.cache_k, model.cache_v = [l["k"] for l in model.cache.layers], [l["v"] for l in model.cache.layers]
+                model._kernel_for_batch = {}
+                model.freqs = pkg.rope_table.precompute_freqs_cis(llama.head_dim, P + long, llama.rope_theta, llama.rope_scaled,
+                                                                  scale_factor=llama.rope_scale_factor).to(dev)
+            prompts = torch.randint(0, 128256, (B, P), generator=torch.Generator().manual_seed(7 + rank)).to(dev)
+            model.generate(prompts, short)
+            if (name, B) == ("nibelorn", 64):
+                sampler.mark("t0")
+            prefill = timed(lambda: model.generate(prompts, 1))
+            steps = []
+            for _ in range(3):
+                timing = {}
+                sync_all(world)
+                model.generate(prompts, long, timing=timing)
+                torch.cuda.synchronize()
+                steps.append(timing["events"][0].elapsed_time(timing["events"][1]) / timing["steps"])
+            step = max_over_ranks(sorted(steps)[1], world, dev)
+            if (name, B) == ("nibelorn", 64):
+                sampler.mark("t1")
+                host, back = prompts.cpu().pin_memory(), torch.empty(B, long, dtype=torch.int64).pin_memory()
+
+                def whole():
+                    back.copy_(model.generate(host.to(dev, non_blocking=True), long), non_blocking=True)
+
+                ms = timed(whole)
+                e2e = {"value": B * long * world / ms * 1e3, "unit": "tokens/s", "h2d_bytes_per_step": host.numel() * 8,
+                       "d2h_bytes_per_step": back.numel() * 8, "ms_per_step": ms,
+                       "note": f"one generation of {long} tokens per sequence with its prefill and graph capture"}
+            models[name][f"B={B} prompt={P}"] = {"prefill_ms": prefill, "prefill_tokens_per_s": B * P * world / prefill * 1e3,
+                                                 "decode_ms_per_step": step, "decode_tokens_per_s": B * world / step * 1e3}
+        del model
+        torch.cuda.empty_cache()
+    sampler.stop()
+    head = models["nibelorn"]["B=64 prompt=1024"]
+    return {
+        "metric": "Nibelorn decode tokens/sec", "value": head["decode_tokens_per_s"], "unit": "tokens/s", "n_gpus": world,
+        "steps": long - 2, "warmup": short, "ms_per_step": head["decode_ms_per_step"], "higher_is_better": True, "scaling": "weak",
+        "vs_baseline": None, "dtype": "bf16", "data": "synthetic",
+        "config": {"model": "Nibelorn, random weights: width 2048, 16 layers (latent attention 16 x (128 + 64), rank 512, values 128; "
+                            "differential attention 16 / 4 heads, 2 x 64, values 128), feed-forward 8192, vocabulary 128256",
+                   "beside": "Llama-3 decoder of equal width, depth, feed-forward size and vocabulary (32 / 8 heads of 64)",
+                   "global_batch": 64 * world, "seq_len": 1024, "parallelism": "replicas x%d" % world,
+                   "l2": "weights and cache of a step exceed L2"},
+        "models": models, "kernels": mixer_kernel_table(ext, pkg, dev, latent, differential) if rank == 0 else None,
+        "e2e": e2e,
+        # embedding, 16 x (cache write, attention, two norms, gelu), token choice; the split merges come on top
+        "gpu_launches": (long - 2) * (1 + 16 * 5 + 1), "clocks": sampler.summary(),
+    }
+
+
+def mixer_kernel_table(ext, pkg, dev, latent, differential):
+    """Roofline of every mixer kernel beside the Llama-3 kernel that does the like: fraction of the measured peak each."""
+    mx = pkg.mixers
+    hbm, _ = hbm_peak()
+    peaks = REPO / "MEASURED_PEAKS.json"
+    tensor = float(json.loads(peaks.read_text())["bf16_tflops"]) if peaks.exists() else 1590.0
+    bf16 = dict(dtype=torch.bfloat16, device=dev)
+    table = []
+
+    def us(step, n):
+        run = graph_runner(step, n, dev)
+        run.prepare(n)
+        run(4 * n)
+        times = []
+        for _ in range(5):
+            start, end = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+            torch.cuda.synchronize()
+            start.record()
+            run(8 * n)
+            end.record()
+            torch.cuda.synchronize()
+            times.append(start.elapsed_time(end) * 1e3 / (8 * n))
+        return sorted(times)[2]
+
+    def sets(bytes_each):
+        return int(max(2, min(24, 4e8 // bytes_each + 1)))   # rotating inputs beyond L2
+
+    def row(name, shape, ours, like_name, like):
+        """ours, like: (microseconds, bytes or flops, peak per microsecond)"""
+        frac = [work / t / peak for t, work, peak in (ours, like)]
+        table.append({"kernel": name, "shape": shape, "us": ours[0], "frac": frac[0], "like": like_name, "like_us": like[0],
+                      "like_frac": frac[1], "frac_over_like": frac[0] / frac[1]})
+        torch.cuda.empty_cache()
+
+    byte, flop = hbm * 1e3, tensor * 1e6   # bytes, flops per microsecond
+    C, R, H, D, V = latent.kv_rank, latent.rot_dim, latent.heads, latent.dim, latent.vdim
+    G, d, Hd, Vd = differential.kv_heads, differential.dim, differential.heads, differential.vdim
+
+    def flash(B, S, Dh):
+        n = sets(B * S * 8 * Dh * 4)
+        k, v = ([torch.randn(B, S, 8, Dh, **bf16).transpose(1, 2) for _ in range(n)] for _ in range(2))
+        q = torch.randn(B, 1, 32, Dh, **bf16).transpose(1, 2)
+        return us(lambda i: ext.flash_attention_decode(q, k[i], v[i]), n), B * S * 8 * Dh * 4, byte
+
+    for B, S in ((64, 1024), (64, 2048), (8, 8192), (1, 65536)):
+        pos = torch.full((B,), S - 1, dtype=torch.int32, device=dev)
+        n = sets(B * S * (C + R) * 2)
+        rows = [torch.randn(B, S, 1, C + R, **bf16) for _ in range(n)]
+        q, o = torch.randn(B, 1, H, C + R, **bf16), torch.empty(H, B, 1, C, **bf16).permute(1, 2, 0, 3)
+        t = us(lambda i: mx.attention(q[..., :C], rows[i][..., :C], rows[i][..., :C], o, pos, qb=q[..., C:], kb=rows[i][..., C:],
+                                      scale=latent.scale), n)
+        del rows
+        like = flash(B, S, 64)
+        row("latent decode attention", f"B={B} keys={S}", (t, B * S * (C + R) * 2, byte), "flash_decode 32/8 x 64", like)
+        n = sets(B * S * G * (2 * d + Vd) * 2)
+        k, v = [torch.randn(B, S, G, 2 * d, **bf16) for _ in range(n)], [torch.randn(B, S, G, Vd, **bf16) for _ in range(n)]
+        q, o, gate = torch.randn(B, 1, Hd, 2 * d, **bf16), torch.empty(B, 1, Hd, Vd, **bf16), torch.randn(B, 1, Hd, **bf16)
+        t = us(lambda i: mx.attention(q, k[i], v[i], o, pos, maps=2, scale=differential.scale, softcap=50.0, temp_coef=0.3,
+                                      temp_every=256.0, gate=gate, lambda_=0.5, post=0.5, eps=1e-5), n)
+        del k, v
+        row("differential decode attention", f"B={B} keys={S}", (t, B * S * G * (2 * d + Vd) * 2, byte), "flash_decode 32/8 x 64", like)
+    for B, T in ((4, 2048), (1, 8192)):
+        pos, pairs = torch.zeros(B, dtype=torch.int32, device=dev), B * T * (T + 1) / 2
+
+        def prefill(Dh):
+            q = torch.randn(B, T, 32, Dh, **bf16).transpose(1, 2)
+            k, v = ([torch.randn(B, T, 8, Dh, **bf16).transpose(1, 2) for _ in range(4)] for _ in range(2))
+            return us(lambda i: ext.prefill_attention(q, k[i], v[i]), 4), 4 * 32 * pairs * Dh, flop
+
+        q = torch.randn(B, T, H, D + R, **bf16)
+        kv, k_rot = [torch.randn(B, T, H * (D + V), **bf16) for _ in range(4)], torch.randn(B, T, 1, R, **bf16)
+        o = torch.empty(B, T, H, V, **bf16)
+        t = us(lambda i: mx.attention(q[..., :D], kv[i][..., :H * D].view(B, T, H, D), kv[i][..., H * D:].view(B, T, H, V), o, pos,
+                                      qb=q[..., D:], kb=k_rot.expand(B, T, H, R), scale=latent.scale, start_pos=0, variant=mx.TC), 4)
+        del kv
+        row("latent prefill attention", f"B={B} T={T}", (t, 2 * H * pairs * (D + R + V), flop), "prefill_attention 32/8 x 128", prefill(128))
+        q, gate, o = torch.randn(B, T, Hd, 2 * d, **bf16), torch.randn(B, T, Hd, **bf16), torch.empty(B, T, Hd, Vd, **bf16)
+        k, v = [torch.randn(B, T, G, 2 * d, **bf16) for _ in range(4)], [torch.randn(B, T, G, Vd, **bf16) for _ in range(4)]
+        t = us(lambda i: mx.attention(q, k[i], v[i], o, pos, maps=2, scale=differential.scale, softcap=50.0, temp_coef=0.3,
+                                      temp_every=256.0, gate=gate, lambda_=0.5, post=0.5, eps=1e-5, start_pos=0, variant=mx.TC), 4)
+        del k, v
+        row("differential prefill attention", f"B={B} T={T}", (t, 4 * Hd * pairs * (d + Vd), flop), "prefill_attention 32/8 x 64", prefill(64))
+    E, F_ = 2048, 8192
+    for B, T in ((64, 1), (4, 2048)):
+        N = B * T
+        n = sets(N * E * 12)
+        w, b, wb = torch.ones(E, device=dev), torch.zeros(E, device=dev), torch.ones(E, **bf16)
+        x, y = [torch.randn(N, E, device=dev) for _ in range(n)], [torch.randn(N, E, **bf16) for _ in range(n)]
+        t = us(lambda i: mx.add_dyn_tanh(y[i], x[i], w, b, 0.5), n)
+        xb = [torch.randn(N, E, **bf16) for _ in range(n)]
+        row("add_dyn_tanh", f"{N} x {E}", (t, N * E * 12, byte), "add_rms_norm",
+            (us(lambda i: ext.add_rms_norm(y[i], xb[i], wb, 1e-5), n), N * E * 8, byte))
+        del x, y, xb
+        n = sets(N * F_ * 4)
+        z, gu = [torch.randn(N, F_, **bf16) for _ in range(n)], [torch.randn(N, 2 * F_, **bf16) for _ in range(n)]
+        t = us(lambda i: mx.gelu_(z[i]), n)
+        row("gelu", f"{N} x {F_}", (t, N * F_ * 4, byte), "silu_mul",
+            (us(lambda i: ext.silu_mul(gu[i][:, :F_], gu[i][:, F_:]), n), N * F_ * 6, byte))
+        del z, gu
+        n, pos = sets(N * 3072 * 2), torch.zeros(B, dtype=torch.int32, device=dev)
+        qkv = [torch.randn(B, T, 48 * 64, **bf16) for _ in range(n)]
+        ck, cv = torch.zeros(B, T + 8, 8, 64, **bf16), torch.zeros(B, T + 8, 8, 64, **bf16)
+        freqs = pkg.rope_table.precompute_freqs_cis(64, T + 8).to(dev)
+        like = (us(lambda i: ext.rot_embed_kv_cache(qkv[i], freqs, ck, cv, 0, 32, 8, positions=pos), n), N * 48 * 64 * 4, byte)
+        del qkv
+        qd = [torch.randn(B, T, H * (D + R) + C + R, **bf16) for _ in range(n)]
+        cache, rot = torch.zeros(B, T + 8, C + R, **bf16), pkg.rope_table.rotation_table(R, T + 8, 1e4).to(dev)
+        nw = torch.ones(C, device=dev)
+        t = us(lambda i: mx.latent_cache(qd[i], rot, nw, 1e-5, cache, pos, H, D, R, C), n)
+        row("latent_cache", f"{N} tokens", (t, N * (H * R + C + R) * 4, byte), "rot_embed_kv_cache", like)
+        pk = [torch.randn(B, T, 2 * Hd * d + G * (2 * d + Vd) + Hd, **bf16) for _ in range(n)]
+        ck, cv = torch.zeros(B, T + 8, G, 2 * d, **bf16), torch.zeros(B, T + 8, G, Vd, **bf16)
+        t = us(lambda i: mx.kv_cache_write(pk[i], 2 * Hd * d, 2 * (Hd + G) * d, ck, cv, pos), n)
+        row("kv_cache_write", f"{N} tokens", (t, N * G * (2 * d + Vd) * 4, byte), "rot_embed_kv_cache", like)
+    return table
 
 
 def time_sampling_step(ext, dev, B, vocab):

@@ -122,24 +122,32 @@ latent_cache_vec_kernel(__nv_bfloat16* __restrict__ qd, const float* __restrict_
   pdl_launch_dependents();
   const long long row = blockIdx.x;
   const int b = (int)(row / p.T), t = (int)(row % p.T), tid = threadIdx.x;
+  // the row's own loads do not wait for the position
   const long long pos = (long long)positions[b] + t;
-  if (pos < 0 || pos >= p.table_rows || pos >= p.cache_len) return;
   __nv_bfloat16* r = qd + row * p.qd_stride;
-  const int head = p.dim + p.rot, half = p.rot / 2, per_head = half / 8;   // vector pairs per head
+  const int head = p.dim + p.rot, half = p.rot / 2, per_head = half / 8, tasks = (p.H + 1) * per_head;   // pairs of vectors
   const __nv_bfloat16* down = r + (long long)p.H * head;
-  __nv_bfloat16* dst = cache + b * p.cache_sb + pos * p.cache_st;
-  const float* cs = table + pos * p.rot;
   uint4 c[VPT];
 #pragma unroll
   for (int i = 0; i < VPT; ++i) {
     const int v = tid + i * kLatentThreads;
     c[i] = v * 8 < p.rank ? *reinterpret_cast<const uint4*>(down + v * 8) : make_uint4(0, 0, 0, 0);
   }
-  for (int i = tid; i < (p.H + 1) * per_head; i += kLatentThreads) {
+  auto load_pair = [&](int i, uint4& u, uint4& v) {
     const int n = i / per_head, j = (i - n * per_head) * 8;
     const __nv_bfloat16* src = n < p.H ? r + (long long)n * head + p.dim : down + p.rank;
+    u = *reinterpret_cast<const uint4*>(src + j);
+    v = *reinterpret_cast<const uint4*>(src + j + half);
+  };
+  uint4 uv = make_uint4(0, 0, 0, 0), vv = uv;
+  if (tid < tasks) load_pair(tid, uv, vv);
+  if (pos < 0 || pos >= p.table_rows || pos >= p.cache_len) return;
+  __nv_bfloat16* dst = cache + b * p.cache_sb + pos * p.cache_st;
+  const float* cs = table + pos * p.rot;
+  for (int i = tid; i < tasks; i += kLatentThreads) {
+    const int n = i / per_head, j = (i - n * per_head) * 8;
     __nv_bfloat16* to = n < p.H ? r + (long long)n * head + p.dim : dst + p.rank;
-    const uint4 uv = *reinterpret_cast<const uint4*>(src + j), vv = *reinterpret_cast<const uint4*>(src + j + half);
+    if (i != tid) load_pair(i, uv, vv);
     float u[8], v[8], x[8], y[8];
     unpack8(uv, u);
     unpack8(vv, v);
@@ -179,11 +187,101 @@ latent_cache_vec_kernel(__nv_bfloat16* __restrict__ qd, const float* __restrict_
   }
 }
 
-// ---- k and v columns of a projection row into the caches ------------------------------------------------------
-// A thread copies kCopies accesses of VEC elements, all loaded before the first is stored.
-constexpr int kCopies = 4;
+// Many tokens: a warp per token, no barrier, the token's latent and its first 32 * kPairsAhead vector pairs in flight at once.
+constexpr int kPairsAhead = 3;
 
-template <typename S, int VEC>
+template <int VPL>
+__global__ void __launch_bounds__(256)
+latent_cache_rows_kernel(__nv_bfloat16* __restrict__ qd, const float* __restrict__ table, const float* __restrict__ nw,
+                         __nv_bfloat16* __restrict__ cache, const int* __restrict__ positions, const LatentRow p, long long rows) {
+  pdl_wait();
+  pdl_launch_dependents();
+  const int lane = threadIdx.x & 31;
+  const long long row = (long long)blockIdx.x * 8 + (threadIdx.x >> 5);
+  if (row >= rows) return;
+  const int b = (int)(row / p.T), t = (int)(row - (long long)b * p.T);
+  const long long pos = (long long)positions[b] + t;
+  __nv_bfloat16* r = qd + row * p.qd_stride;
+  const int head = p.dim + p.rot, half = p.rot / 2, per_head = half / 8, tasks = (p.H + 1) * per_head;
+  const __nv_bfloat16* down = r + (long long)p.H * head;
+  uint4 c[VPL], u[kPairsAhead], v[kPairsAhead];
+#pragma unroll
+  for (int i = 0; i < VPL; ++i) {
+    const int x = lane + 32 * i;
+    c[i] = x * 8 < p.rank ? ld_stream16(down + x * 8) : make_uint4(0, 0, 0, 0);
+  }
+  auto source = [&](int i) {
+    const int n = i / per_head, j = (i - n * per_head) * 8;
+    return (n < p.H ? r + (long long)n * head + p.dim : const_cast<__nv_bfloat16*>(down) + p.rank) + j;
+  };
+  auto load = [&](int i0) {
+#pragma unroll
+    for (int k = 0; k < kPairsAhead; ++k) {
+      const int i = i0 + lane + 32 * k;
+      if (i < tasks) {
+        const __nv_bfloat16* src = source(i);
+        u[k] = *reinterpret_cast<const uint4*>(src);
+        v[k] = *reinterpret_cast<const uint4*>(src + half);
+      }
+    }
+  };
+  load(0);
+  if (pos < 0 || pos >= p.table_rows || pos >= p.cache_len) return;
+  __nv_bfloat16* dst = cache + b * p.cache_sb + pos * p.cache_st;
+  const float* cs = table + pos * p.rot;
+  float ss = 0.f;
+#pragma unroll
+  for (int i = 0; i < VPL; ++i) {
+    float f[8];
+    unpack8(c[i], f);
+#pragma unroll
+    for (int k = 0; k < 8; ++k) ss = fmaf(f[k], f[k], ss);
+  }
+  ss = group_sum<32>(ss);
+  const float inv = __frsqrt_rn(__fadd_rn(__fdiv_rn(ss, (float)p.rank), p.eps));
+#pragma unroll
+  for (int i = 0; i < VPL; ++i) {
+    const int x = lane + 32 * i;
+    if (x * 8 < p.rank) {
+      float f[8];
+      unpack8(c[i], f);
+      const float4 w0 = __ldg(reinterpret_cast<const float4*>(nw + x * 8)), w1 = __ldg(reinterpret_cast<const float4*>(nw + x * 8 + 4));
+      const float w[8] = {w0.x, w0.y, w0.z, w0.w, w1.x, w1.y, w1.z, w1.w};
+#pragma unroll
+      for (int k = 0; k < 8; ++k) f[k] = f[k] * inv * w[k];
+      *reinterpret_cast<uint4*>(dst + x * 8) = pack8(f);
+    }
+  }
+  for (int i0 = 0;; ) {
+#pragma unroll
+    for (int k = 0; k < kPairsAhead; ++k) {
+      const int i = i0 + lane + 32 * k;
+      if (i >= tasks) continue;
+      const int n = i / per_head, j = (i - n * per_head) * 8;
+      __nv_bfloat16* to = n < p.H ? source(i) : dst + p.rank + j;
+      float a[8], d[8], x[8], y[8];
+      unpack8(u[k], a);
+      unpack8(v[k], d);
+#pragma unroll
+      for (int q = 0; q < 8; q += 2) {
+        const float4 f = __ldg(reinterpret_cast<const float4*>(cs + 2 * (j + q)));
+        x[q] = a[q] * f.x - d[q] * f.y;
+        y[q] = d[q] * f.x + a[q] * f.y;
+        x[q + 1] = a[q + 1] * f.z - d[q + 1] * f.w;
+        y[q + 1] = d[q + 1] * f.z + a[q + 1] * f.w;
+      }
+      *reinterpret_cast<uint4*>(to) = pack8(x);
+      *reinterpret_cast<uint4*>(to + half) = pack8(y);
+    }
+    i0 += 32 * kPairsAhead;
+    if (i0 >= tasks) break;
+    load(i0);
+  }
+}
+
+// ---- k and v columns of a projection row into the caches ------------------------------------------------------
+// A thread copies COPIES accesses of VEC elements, all loaded before the first is stored.
+template <typename S, int VEC, int COPIES>
 __global__ void __launch_bounds__(128)
 kv_cache_write_kernel(const S* __restrict__ src, long long stride, long long k_col, int k_width, long long v_col, int v_width,
                       S* __restrict__ ck, long long k_sb, long long k_st, S* __restrict__ cv, long long v_sb, long long v_st,
@@ -192,12 +290,12 @@ kv_cache_write_kernel(const S* __restrict__ src, long long stride, long long k_c
   pdl_launch_dependents();
   using R = typename Raw<VEC * sizeof(S)>::type;
   const unsigned per_row = (k_width + v_width) / VEC;
-  R data[kCopies];
-  S* to[kCopies];
+  R data[COPIES];
+  S* to[COPIES];
 #pragma unroll
-  for (int u = 0; u < kCopies; ++u) {
+  for (int u = 0; u < COPIES; ++u) {
     to[u] = nullptr;
-    const long long id = ((long long)blockIdx.x * kCopies + u) * 128 + threadIdx.x;
+    const long long id = ((long long)blockIdx.x * COPIES + u) * 128 + threadIdx.x;
     if (id >= (long long)rows * per_row) continue;
     const long long row = per_row * (long long)rows <= 0xffffffffLL ? (unsigned)id / per_row : id / per_row;
     const int i = (int)(id - row * per_row) * VEC, b = (int)(row / T), t = (int)(row % T);
@@ -208,7 +306,7 @@ kv_cache_write_kernel(const S* __restrict__ src, long long stride, long long k_c
     to[u] = is_k ? ck + b * k_sb + pos * k_st + i : cv + b * v_sb + pos * v_st + (i - k_width);
   }
 #pragma unroll
-  for (int u = 0; u < kCopies; ++u)
+  for (int u = 0; u < COPIES; ++u)
     if (to[u]) *reinterpret_cast<R*>(to[u]) = data[u];
 }
 
@@ -296,6 +394,14 @@ int l3ci_latent_cache(void* qd, int64_t qd_stride, const float* table, int64_t t
   const bool vec = dtype == L3CI_BF16 && rank % 8 == 0 && rot_dim % 16 == 0 && dim % 8 == 0 && qd_stride % 8 == 0 && cache_sb % 8 == 0 &&
                    cache_st % 8 == 0 && rank <= 8 * kLatentVecs * kLatentThreads && aligned16(qd) && aligned16(cache) &&
                    aligned16(table) && aligned16(norm_weight);
+  if (vec && rank <= 1024 && rows >= 16LL * sm_count()) {
+    auto go = [&](auto kernel) -> int {
+      L3CI_LAUNCH("latent_cache_rows_kernel", kernel, dim3((unsigned)((rows + 7) / 8)), dim3(256), 0, s, static_cast<__nv_bfloat16*>(qd),
+                  table, norm_weight, static_cast<__nv_bfloat16*>(cache), positions, p, rows);
+      return L3CI_OK;
+    };
+    return rank <= 512 ? go(latent_cache_rows_kernel<2>) : go(latent_cache_rows_kernel<4>);
+  }
   if (vec) {
     auto go = [&](auto kernel) -> int {
       L3CI_LAUNCH("latent_cache_vec_kernel", kernel, dim3((unsigned)rows), dim3(kLatentThreads), 0, s, static_cast<__nv_bfloat16*>(qd),
@@ -331,15 +437,16 @@ int l3ci_kv_cache_write(const void* src, int64_t src_stride, int64_t k_col, int6
     constexpr int kVec = 16 / sizeof(S);
     const int64_t all = src_stride | k_col | k_width | v_col | v_width | k_sb | k_st | v_sb | v_st;
     const bool v = all % kVec == 0 && aligned16(src) && aligned16(cache_k) && aligned16(cache_v);
-    auto go = [&](auto kernel, int width) -> int {
-      const long long units = rows * ((k_width + v_width) / width), per_cta = 128LL * kCopies;
+    auto go = [&](auto kernel, int width, int copies) -> int {
+      const long long units = rows * ((k_width + v_width) / width), per_cta = 128LL * copies;
       if ((units + per_cta - 1) / per_cta > 0x7fffffffLL) return fail(L3CI_ERR_INVALID, "kv_cache_write: too much");
       L3CI_LAUNCH("kv_cache_write_kernel", kernel, dim3((unsigned)((units + per_cta - 1) / per_cta)), dim3(128), 0, s, static_cast<const S*>(src), (long long)src_stride,
                   (long long)k_col, (int)k_width, (long long)v_col, (int)v_width, static_cast<S*>(cache_k), (long long)k_sb,
                   (long long)k_st, static_cast<S*>(cache_v), (long long)v_sb, (long long)v_st, (long long)cache_len, positions, T, (int)rows);
       return L3CI_OK;
     };
-    return v ? go(kv_cache_write_kernel<S, kVec>, kVec) : go(kv_cache_write_kernel<S, 1>, 1);
+    if (!v) return go(kv_cache_write_kernel<S, 1, 1>, 1, 1);
+    return rows < 1024 ? go(kv_cache_write_kernel<S, kVec, 1>, kVec, 1) : go(kv_cache_write_kernel<S, kVec, 4>, kVec, 4);
   };
   return dtype == L3CI_BF16 ? typed(__nv_bfloat16{}) : typed(float{});
 }

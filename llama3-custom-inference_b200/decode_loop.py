@@ -151,11 +151,12 @@ class DecodeLoop:
     # ---- generation ---------------------------------------------------------------------------------------
     @torch.inference_mode()
     def generate(self, prompts: torch.Tensor, max_gen_len: int, use_graph: bool = True, temperature: float = 0.0,
-                 top_p: float = 0.9, seed: int = 0) -> torch.Tensor:
+                 top_p: float = 0.9, seed: int = 0, timing: Optional[dict] = None) -> torch.Tensor:
         """prompts int64 [B, P] (equal lengths, on the device).  Returns the generated tokens int64
         [B, max_gen_len].  With `use_graph` one decode step is captured in a CUDA graph and replayed.
         `temperature` 0 is greedy decoding (model.py:370-371); a positive temperature draws every token from the
-        top-p nucleus of softmax(logits / temperature) (model.py:367-369), reproducibly for a given `seed`."""
+        top-p nucleus of softmax(logits / temperature) (model.py:367-369), reproducibly for a given `seed`.  `timing` (a
+        dict) receives "events" (two CUDA events around the replayed steps) and "steps" (their number)."""
         B, P = prompts.shape
         assert B <= self.max_batch and P + max_gen_len <= self.max_len
         dev = self.device
@@ -203,8 +204,13 @@ class DecodeLoop:
                 with torch.cuda.graph(graph, stream=side):
                     step()
                 # the capture did not run the step: replay it for every remaining token
+                if timing is not None:
+                    timing.update(events=[torch.cuda.Event(enable_timing=True) for _ in range(2)], steps=n_steps)
+                    timing["events"][0].record(side)
                 for _ in range(n_steps):
                     graph.replay()
+                if timing is not None:
+                    timing["events"][1].record(side)
         torch.cuda.current_stream(dev).wait_stream(side)
         self._graph = graph
         return out

@@ -99,10 +99,33 @@ def test_latent_cache_rows(pkg, device, dtype, H, D, R, C):
     assert bool((untouched == 7.0).all()) and bool((cache[..., C + R:] == 7.0).all())
 
 
+@pytest.mark.parametrize("H,D,R,C", [(3, 24, 16, 40), (16, 128, 64, 512), (20, 32, 96, 768)])
+def test_latent_cache_rows_of_many_tokens(pkg, device, H, D, R, C):
+    """The warp-per-token form: enough tokens to take it, the last ones beyond the cache."""
+    B, T, L, base, eps = 2, 1500, 1600, 500.0, 1e-5
+    W = H * (D + R) + C + R
+    qd, nw = rand(B, T, W, seed=9), rand(C, seed=10, dtype=F32)
+    cache = torch.full((B, L, C + R), 7.0, dtype=BF16, device=device)
+    positions = torch.tensor([0, 150], dtype=torch.int32, device=device)
+    dq = qd.to(device).clone()
+    pkg.mixers.latent_cache(dq, pkg.rope_table.rotation_table(R, L, base).to(device), nw.to(device), eps, cache, positions, H, D, R, C)
+    for b, p0, n in ((0, 0, T), (1, 150, L - 150)):
+        pos, rows = torch.arange(p0, p0 + n), qd[b, :n].double()
+        q, down = rows[:, :H * (D + R)].view(n, H, D + R), rows[:, H * (D + R):]
+        got = dq[b, :, :H * (D + R)].view(T, H, D + R)
+        assert torch.equal(got[..., :D].cpu(), qd[b, :, :H * (D + R)].view(T, H, D + R)[..., :D])
+        close(got[:n, :, D:], ref.rotate_half(q[..., D:], pos, base), BF16, "q")
+        assert torch.equal(got[n:, :, D:].cpu(), qd[b, n:, :H * (D + R)].view(T - n, H, D + R)[..., D:])
+        close(cache[b, p0:p0 + n, :C], ref.rms(down[:, :C], eps) * nw.double(), BF16, "latent")
+        close(cache[b, p0:p0 + n, C:], ref.rotate_half(down[:, C:], pos, base), BF16, "k")
+    assert bool((cache[0, T:] == 7.0).all()) and bool((cache[1, :150] == 7.0).all())
+
+
 @pytest.mark.parametrize("dtype", [BF16, F32])
 @pytest.mark.parametrize("G,D,V", [(2, 8, 24), (3, 5, 7)])
-def test_kv_cache_write(pkg, device, dtype, G, D, V):
-    B, T, L = 2, 4, 20
+@pytest.mark.parametrize("T", [4, 700])
+def test_kv_cache_write(pkg, device, dtype, G, D, V, T):
+    B, L = 2, T + 16
     src = rand(B, T, 16 + G * (2 * D + V) + 8, seed=11, dtype=dtype).to(device)
     k = torch.zeros(B, L, G, 2 * D, dtype=dtype, device=device)
     v = torch.zeros(B, L, G, V, dtype=dtype, device=device)
