@@ -1055,10 +1055,9 @@ def bench_nibelorn(args, ext, pkg, dev, rank, world):
     llama = dl.DecoderConfig()
     short, long = 17, 129
     shapes = ((64, 1024), (8, 4096), (1, 8192))
-    makers = {
-        "nibelorn": lambda B, L: nb.NibelornDecoder(ext, cfg, dev, B, L, weights=nb.init_weights(cfg, 42 + rank, dev)),
-        "llama3": lambda B, L: dl.Llama3Decoder(ext, llama, dev, B, L, seed=42 + rank),
-    }
+    weights = {"nibelorn": lambda: nb.init_weights(cfg, 42 + rank, dev),
+               "llama3": lambda: {k: v.to(dev) for k, v in dl.init_weights(llama, 42 + rank).items()}}
+    decoders = {"nibelorn": (nb.NibelornDecoder, cfg), "llama3": (dl.Llama3Decoder, llama)}
 
     def timed(fn, repeats=3):
         times = []
@@ -1075,21 +1074,11 @@ def bench_nibelorn(args, ext, pkg, dev, rank, world):
     sampler = ClockSampler(dev.index or 0)
     sampler.start()
     models, e2e = {}, None
-    for name, make in makers.items():
-        model = make(64, max(64 * (1024 + long), 8 * (4096 + long), 8192 + long) // 64 + 1)
+    for name, (decoder, config) in decoders.items():
+        w = weights[name]()
         models[name] = {}
         for B, P in shapes:
-            # the same weights behind a cache of this shape: slots and length follow the batch
-            model.cache = pkg.kv_cache.StaticCache([{n: tuple(t.shape[2:]) for n, t in layer.items()} for layer in model.cache.layers],
-                                                   B, P + long, model.dtype, dev)
-            model.max_batch, model.max_len = B, P + long
-            if name == "nibelorn":
-                model._tables = {k: pkg.rope_table.rotation_table(k[0], P + long, k[1]).to(dev) for k in model._tables}
-            else:
-                model.cache_k, model.cache_v = [l["k"] for l in model.cache.layers], [l["v"] for l in model.cache.layers]
-                model._kernel_for_batch = {}
-                model.freqs = pkg.rope_table.precompute_freqs_cis(llama.head_dim, P + long, llama.rope_theta, llama.rope_scaled,
-                                                                  scale_factor=llama.rope_scale_factor).to(dev)
+            model = decoder(ext, config, dev, B, P + long, weights=dict(w))
             prompts = torch.randint(0, 128256, (B, P), generator=torch.Generator().manual_seed(7 + rank)).to(dev)
             model.generate(prompts, short)
             if (name, B) == ("nibelorn", 64):
@@ -1116,8 +1105,9 @@ def bench_nibelorn(args, ext, pkg, dev, rank, world):
                        "note": f"one generation of {long} tokens per sequence with its prefill and graph capture"}
             models[name][f"B={B} prompt={P}"] = {"prefill_ms": prefill, "prefill_tokens_per_s": B * P * world / prefill * 1e3,
                                                  "decode_ms_per_step": step, "decode_tokens_per_s": B * world / step * 1e3}
-        del model
-        torch.cuda.empty_cache()
+            del model
+            torch.cuda.empty_cache()
+        del w
     sampler.stop()
     head = models["nibelorn"]["B=64 prompt=1024"]
     return {
