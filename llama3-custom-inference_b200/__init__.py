@@ -11,12 +11,13 @@ The directory name is not a Python identifier, so load this package by path, e.g
 Contents:
   build.py        in-tree build of lib/libl3ci_b200.so, lib/libl3ci_mixers.so and custom_kernels/custom_kernels_extension.so
   capi.py         ctypes binding of the C ABI (include/l3ci_b200.h) over torch device tensors
-  mixers.py       the same for include/l3ci_mixers.h (latent and differential attention, dynamic-tanh norm, gelu)
+  mixers.py       the same for include/l3ci_mixers.h (attention kinds, linear recurrences, experts, norms, activations)
   rope_table.py   rotary table with the Llama-3 frequency scaling as parameters (model.py:27-60)
   sharding.py     partition of a decode batch / a long KV sequence over the GPUs of one box
   decode_loop.py  what decoders share (cache, requests, generation) and the Llama-3 decoder (end-to-end tokens/s harness)
   kv_cache.py     static per-layer caches and the requests that hold their slots
   nibelorn.py     the Nibelorn decoder (latent and differential attention)
+  rupotar.py      the Rupotar decoder (windowed attention, two linear recurrences, experts, looped layers)
   models.py       registry: config.json -> configuration, weights, decoder;  checkpoint.py reads a model folder
   custom_kernels/ the torch extension module; put this package directory on sys.path and the
                   reference's `from custom_kernels import custom_kernels_extension` (model.py:23)
@@ -52,4 +53,4 @@ def extension():
     return importlib.import_module("custom_kernels.custom_kernels_extension")
 
 
-from . import capi, checkpoint, decode_loop, kv_cache, mixers, models, nibelorn, rope_table, sharding  # noqa: E402,F401
+from . import capi, checkpoint, decode_loop, kv_cache, mixers, models, nibelorn, rope_table, rupotar, sharding  # noqa: E402,F401

@@ -42,7 +42,7 @@ NVCC_FLAGS = [
 ]
 CUDA_SOURCES = ["host_common.cu", "rms_norm.cu", "rope.cu", "flash_decode.cu", "flash_decode_small.cu", "lse_merge.cu", "greedy_step.cu", "top_p_step.cu", "prefill_attention.cu", "prefill_attention_tc.cu"]
 
-MIXER_SOURCES = ["host_common.cu", "mixer_parts.cu", "mixer_attention.cu", "mixer_attention_mma.cu", "mixer_attention_tc.cu"]
+MIXER_SOURCES = ["host_common.cu", "mixer_parts.cu", "mixer_attention.cu", "mixer_attention_mma.cu", "mixer_attention_tc.cu", "mixer_residual.cu", "mixer_recurrent.cu", "mixer_moe.cu", "mixer_moe_tc.cu"]
 
 
 def _nvcc() -> str:

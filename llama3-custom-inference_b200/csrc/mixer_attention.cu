@@ -38,7 +38,10 @@ __global__ void __launch_bounds__(kRowThreads) mixer_rows_kernel(const l3ci_mixe
   pdl_launch_dependents();
   const int t = blockIdx.x, h = blockIdx.y, b = blockIdx.z, g = h / (a.H / a.G), tid = threadIdx.x;
   const int pos = a.positions[b] + t;
-  const int keys = min(pos + 1, a.n_keys);
+  // the keys in sight: the first `kept` ones, then those from `lo` on
+  const int lo = window_start(pos, a.window), kept = min(a.keep_first, lo);
+  const int keys = kept + max(0, min(pos + 1, a.n_keys) - lo);
+  const float slope = head_slope(a.bias_range, h, a.H);
   float* qs = sh;  // [MAPS][Da + Db]
   const int dk = a.Da + a.Db;
   const S* qa = static_cast<const S*>(a.qa) + b * a.qa_sb + t * a.qa_st + h * a.qa_sh;
@@ -55,17 +58,18 @@ __global__ void __launch_bounds__(kRowThreads) mixer_rows_kernel(const l3ci_mixe
   float acc[MAPS][kRowCols], m_run[MAPS], l_run[MAPS];
 #pragma unroll
   for (int m = 0; m < MAPS; ++m) {
-    m_run[m] = -INFINITY;
-    l_run[m] = 0.f;
+    m_run[m] = a.sink ? 0.f : -INFINITY;
+    l_run[m] = a.sink ? 1.f : 0.f;
 #pragma unroll
     for (int c = 0; c < kRowCols; ++c) acc[m][c] = 0.f;
   }
   for (int j0 = 0; j0 < keys; j0 += kRowThreads) {
-    const int j = j0 + tid;
+    const bool seen = j0 + tid < keys;
+    const int j = j0 + tid < kept ? j0 + tid : lo + j0 + tid - kept;
 #pragma unroll
     for (int m = 0; m < MAPS; ++m) {
       float s = -INFINITY;
-      if (j < keys) {
+      if (seen) {
         const S* kr = ka + j * a.ka_st + m * a.Da;
         s = 0.f;
         for (int d = 0; d < a.Da; ++d) s = fmaf(qs[m * dk + d], to_f32(kr[d]), s);
@@ -73,9 +77,10 @@ __global__ void __launch_bounds__(kRowThreads) mixer_rows_kernel(const l3ci_mixe
         for (int d = 0; d < a.Db; ++d) s = fmaf(qs[m * dk + a.Da + d], to_f32(kr2[d]), s);
         s *= scale;
         if (a.softcap > 0.f) s = a.softcap * tanhf(s / a.softcap);
+        s -= slope * (float)(pos - j);
       }
       const float mx = fmaxf(m_run[m], cta_max(s, red));
-      const float p = j < keys ? expf(s - mx) : 0.f;
+      const float p = seen ? expf(s - mx) : 0.f;
       const float alpha = m_run[m] == -INFINITY ? 0.f : expf(m_run[m] - mx);
       m_run[m] = mx;
       l_run[m] = fmaf(l_run[m], alpha, cta_sum(p, red, kRowThreads / kWarp));
@@ -90,7 +95,8 @@ __global__ void __launch_bounds__(kRowThreads) mixer_rows_kernel(const l3ci_mixe
       const int col = tid + c * kRowThreads;
       if (col >= a.Dv) continue;
       for (int i = 0; i < n; ++i) {
-        const float x = to_f32(v[(j0 + i) * a.v_st + col]);
+        const int at = j0 + i < kept ? j0 + i : lo + j0 + i - kept;
+        const float x = to_f32(v[at * a.v_st + col]);
 #pragma unroll
         for (int m = 0; m < MAPS; ++m) acc[m][c] = fmaf(pk[m][i], x, acc[m][c]);
       }
@@ -134,6 +140,9 @@ int validate(const l3ci_mixer_attn_args* a) {
       a->Dv <= 0 || a->n_keys < 0 || (a->dtype != L3CI_BF16 && a->dtype != L3CI_F32) || a->variant < 0 || a->variant > 3)
     return fail(L3CI_ERR_INVALID, "mixer_attention: bad size B=%d T=%d H=%d G=%d maps=%d Da=%d Db=%d Dv=%d", a->B, a->T, a->H, a->G,
                 a->maps, a->Da, a->Db, a->Dv);
+  if (a->window < 0 || a->keep_first < 0 || !(a->bias_range >= 0.f)) return fail(L3CI_ERR_INVALID, "mixer_attention: window=%d keep_first=%d", a->window, a->keep_first);
+  if (a->maps == 2 && (a->window || a->sink || a->bias_range > 0.f))
+    return fail(L3CI_ERR_UNSUPPORTED, "mixer_attention: two maps take no window, sink or distance bias");
   if (a->maps == 2 && a->Db) return fail(L3CI_ERR_UNSUPPORTED, "mixer_attention: two maps have one key part");
   if (a->B == 0 || a->T == 0) return L3CI_OK;
   if (!a->qa || !a->ka || !a->v || !a->out || !a->positions || (a->Db && (!a->qb || !a->kb)))

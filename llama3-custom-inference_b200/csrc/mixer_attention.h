@@ -21,6 +21,12 @@ int mixer_tc_launch(const l3ci_mixer_attn_args* a);
 __device__ __forceinline__ float query_temperature(int p, float coef, float every) {
   return every > 0.f ? fmaf(coef, logf(floorf(__fdiv_rn((float)(p + 1), every)) + 1.f), 1.f) : 1.f;
 }
+// First key of position p's window (0: no window).
+__device__ __forceinline__ int window_start(int p, int window) { return window > 0 ? max(0, p - window + 1) : 0; }
+// 2^(-range (h + 1) / H): what a head takes off a score per position of distance; range 0: nothing.
+__device__ __forceinline__ float head_slope(float range, int h, int H) {
+  return range > 0.f ? exp2f(-range * (float)(h + 1) / (float)H) : 0.f;
+}
 #endif
 
 }  // namespace l3ci

@@ -139,10 +139,14 @@ mixer_mma_kernel(const __grid_constant__ CUtensorMap kmap, const __grid_constant
   const int pair0 = rb * kPairs, n_pairs = min(kPairs, a.T * p.R - pair0);
   const int pos0 = a.positions[b];
   const int keys = max(0, min(a.n_keys, pos0 + (pair0 + n_pairs - 1) / p.R + 1));
-  const int tiles = (keys + KEYS - 1) / KEYS;
+  // key tiles in sight of any of the unit's rows: those of the kept first keys, then from the first row's window on
+  const int w_tile = window_start(pos0 + pair0 / p.R, a.window) / KEYS;
+  const int kept_tiles = min(w_tile, (a.keep_first + KEYS - 1) / KEYS), skipped = w_tile - kept_tiles;
+  const int tiles = max(0, (keys + KEYS - 1) / KEYS - skipped);
   const int per_split = (tiles + p.splits - 1) / p.splits;
   const int tile0 = split * per_split;
   const int n = max(0, min(tiles, tile0 + per_split) - tile0);
+  auto first_key = [&](int i) { return (tile0 + i + (tile0 + i >= kept_tiles ? skipped : 0)) * KEYS; };   // of the CTA's tile i
   bool ok = true;
 
   if (warp == kWarps) {
@@ -153,7 +157,7 @@ mixer_mma_kernel(const __grid_constant__ CUtensorMap kmap, const __grid_constant
       if (lane == 0) {
         const uint32_t bar = full0 + s * 8, dst = ring + s * stage_bytes;
         mbar_expect_tx(bar, stage_bytes);
-        const int j0 = tile0 * KEYS + i * kStageKeys;
+        const int j0 = first_key(i / Sh::kSub) + i % Sh::kSub * kStageKeys;
         for (int c = 0; c < p.k_boxes; ++c) tma_load_4d(dst + c * kBoxBytes, &kmap, bar, c * 64, j0, g, b, policy);
         for (int c = 0; c < p.v_boxes; ++c) tma_load_4d(dst + (p.k_boxes + c) * kBoxBytes, &vmap, bar, c * 64, j0, g, b, policy);
       }
@@ -218,7 +222,12 @@ mixer_mma_kernel(const __grid_constant__ CUtensorMap kmap, const __grid_constant
   const int limit = pos0 + (pair0 + min(spair, n_pairs - 1)) / p.R;            // last key the row sees
   const float scale = a.scale * query_temperature(limit, a.temp_coef, a.temp_every);
   const float cap = a.softcap, cap_scale = cap > 0.f ? scale / cap : scale * kLog2e, cap_out = cap * kLog2e;
-  float m_run = -INFINITY, l_run = 0.f;
+  const int row_head = g * p.R + (pair0 + min(spair, n_pairs - 1)) % p.R;
+  const float slope = MAPS == 1 ? head_slope(a.bias_range, row_head, a.H) * kLog2e : 0.f;
+  const int row_lo = window_start(limit, a.window);
+  // the sink is a score of 0 that the first split has seen before its first tile
+  const bool sink = MAPS == 1 && a.sink && split == 0;
+  float m_run = sink ? 0.f : -INFINITY, l_run = sink && row_lead ? 1.f : 0.f;
 
   float o[NB][4];
 #pragma unroll
@@ -312,13 +321,14 @@ mixer_mma_kernel(const __grid_constant__ CUtensorMap kmap, const __grid_constant
           for (int e = 0; e < kPer; ++e) v[e] += row[e];
         }
       }
-      const int j0 = (tile0 + i) * KEYS, j = j0 + skey;
+      const int j0 = first_key(i), j = j0 + skey;
       float mx = -INFINITY;
 #pragma unroll
       for (int e = 0; e < kPer; ++e) {
         v[e] *= cap_scale;
         if (cap > 0.f) v[e] = cap_out * tanhf(v[e]);
-        if (j + e > limit || j + e >= keys) v[e] = -INFINITY;
+        if (MAPS == 1) v[e] = fmaf(-slope, (float)(limit - j - e), v[e]);
+        if (j + e > limit || j + e >= keys || (MAPS == 1 && j + e < row_lo && j + e >= a.keep_first)) v[e] = -INFINITY;
         mx = fmaxf(mx, v[e]);
       }
       mx = fmaxf(m_run, group_max<Sh::kRowThreads>(mx));
@@ -585,7 +595,11 @@ MmParams mma_params(const l3ci_mixer_attn_args* a) {
   const int sms = sm_count() > 0 ? sm_count() : 148;
   const long long slots = (long long)sms * per_sm;
   const int keys = a->start_pos >= 0 && a->start_pos + a->T < a->n_keys ? a->start_pos + a->T : a->n_keys;
-  const int tiles = keys > 0 ? (keys + KEYS - 1) / KEYS : 1;
+  int tiles = keys > 0 ? (keys + KEYS - 1) / KEYS : 1;
+  if (a->window > 0) {   // most tiles a unit sees: its window at the worst place, and the kept keys
+    const long long seen = ((long long)a->window + (pairs + p.R - 1) / p.R + KEYS - 1) / KEYS + 1 + (a->keep_first + KEYS - 1) / KEYS;
+    if (seen < tiles) tiles = (int)seen;
+  }
   double best = 0;
   p.splits = 1;
   for (int s = 1; s <= tiles && s <= kMaxSplits; ++s) {

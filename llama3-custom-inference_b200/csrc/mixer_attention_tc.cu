@@ -2,10 +2,11 @@
 // in shared memory (bulk tensor copies, 128-byte swizzle) or tensor memory, accumulators in tensor memory.  The
 // machinery (roles, barriers, lazy reference maximum, P over S, register re-deal) is that of prefill_attention_tc.cu.
 //
-// mixer_tc_kernel<KA, KB, VC>: one map; a query / key vector is two parts (KA and KB boxes of 64 columns, zero-filled
+// mixer_tc_kernel<KA, KB, VC, BIAS>: one map; a query / key vector is two parts (KA and KB boxes of 64 columns, zero-filled
 //   where a part ends), which come from their own tensors: expanded latent attention reads its unrotated keys from the
 //   expansion and the rotated part, shared by the heads, from the cache.  One head per CTA, the two softmax groups take
-//   the even and the odd key tiles and merge at the end.
+//   the even and the odd key tiles and merge at the end.  A window (with kept first keys) skips the tiles no row sees; BIAS
+//   takes a head's distance bias off the scores; a sink is a first score of 0 without a value.
 // mixer_tc_maps_kernel<VC, CAP>: differential attention.  Softmax group e owns map e of a head (its own Q, K, S_e, O_e;
 //   the value tile is loaded once), a persistent grid walks the (head, query block) items longest first, and the output
 //   warpgroup, whose thread holds a row of both maps' outputs, forms the difference, its root mean square over the row
@@ -79,7 +80,7 @@ constexpr float kPolyRange = 0.7f;
 __device__ constexpr float kPoly[5] = {0.999999718f, -0.333303491f, 0.132824955f, -0.0508812513f, 0.0138195432f};
 
 // ---------------------------------------------------------------------------------------------------------------
-template <int KA, int KB, int VC>
+template <int KA, int KB, int VC, bool BIAS>
 __global__ void __launch_bounds__(kOneThreads, 1)
 mixer_tc_kernel(const __grid_constant__ CUtensorMap qamap, const __grid_constant__ CUtensorMap qbmap,
                 const __grid_constant__ CUtensorMap kamap, const __grid_constant__ CUtensorMap kbmap,
@@ -130,7 +131,11 @@ mixer_tc_kernel(const __grid_constant__ CUtensorMap qamap, const __grid_constant
   const int hkv = hq / p.R;
   const int m0 = mb * kRows;
   const int keys = min(p.n_keys, a.start_pos + min(m0 + kRows, a.T));
-  const int n_tiles = (keys + kKeys - 1) / kKeys;
+  // key tiles in sight of any row: those of the kept first keys, then from the first row's window on
+  const int w_tile = window_start(a.start_pos + m0, a.window) / kKeys;
+  const int kept_tiles = min(w_tile, (a.keep_first + kKeys - 1) / kKeys), skipped = w_tile - kept_tiles;
+  const int n_tiles = (keys + kKeys - 1) / kKeys - skipped;
+  auto first_key = [&](int j) { return (j + (j >= kept_tiles ? skipped : 0)) * kKeys; };   // of tile j
   bool ok = true;
 
   if (warp == 0) {
@@ -139,9 +144,9 @@ mixer_tc_kernel(const __grid_constant__ CUtensorMap qamap, const __grid_constant
     const uint64_t policy = l2_evict_first_policy();
     auto load_k = [&](uint32_t dst, uint32_t bar_, int j) {
 #pragma unroll
-      for (int c = 0; c < KA; ++c) tma_load_4d(dst + c * kBox, &kamap, bar_, c * 64, j * kKeys, hkv, b, policy);
+      for (int c = 0; c < KA; ++c) tma_load_4d(dst + c * kBox, &kamap, bar_, c * 64, first_key(j), hkv, b, policy);
 #pragma unroll
-      for (int c = 0; c < KB; ++c) tma_load_4d(dst + (KA + c) * kBox, &kbmap, bar_, c * 64, j * kKeys, p.shared_b ? 0 : hkv, b, policy);
+      for (int c = 0; c < KB; ++c) tma_load_4d(dst + (KA + c) * kBox, &kbmap, bar_, c * 64, first_key(j), p.shared_b ? 0 : hkv, b, policy);
     };
     if (lane == 0) {
       mbar_expect_tx(bar(Q_FULL), kQBytes);
@@ -162,7 +167,7 @@ mixer_tc_kernel(const __grid_constant__ CUtensorMap qamap, const __grid_constant
       if (lane == 0) {
         mbar_expect_tx(bar(V_FULL + s), kVBytes);
 #pragma unroll
-        for (int c = 0; c < VC; ++c) tma_load_4d(v_smem + s * kVBytes + c * kBox, &vmap, bar(V_FULL + s), c * 64, j * kKeys, hkv, b, policy);
+        for (int c = 0; c < VC; ++c) tma_load_4d(v_smem + s * kVBytes + c * kBox, &vmap, bar(V_FULL + s), c * 64, first_key(j), hkv, b, policy);
       }
       __syncwarp();
     }
@@ -219,13 +224,18 @@ mixer_tc_kernel(const __grid_constant__ CUtensorMap qamap, const __grid_constant
     const uint32_t lane_addr = (uint32_t)(q4 * 32) << 16;
     const uint32_t ts = t_s[e] + lane_addr, to = t_o[e] + lane_addr;
     const float scale_log2e = a.scale * kLog2e;
-    float m_ref = -INFINITY, l_run = 0.f;
+    const float slope = BIAS ? head_slope(a.bias_range, hq, a.H) * kLog2e : 0.f;
+    const int row_lo = window_start(limit, a.window);
+    // the sink is a score of 0 that the first group has seen before its first tile
+    float m_ref = a.sink && e == 0 ? 0.f : -INFINITY, l_run = a.sink && e == 0 ? 1.f : 0.f;
     int done = 0;
     for (int j = e; j < n_tiles && ok; j += 2, ++done) {
       if (!mbar_wait_bounded(bar(S_FULL + e), done & 1)) { ok = false; break; }
       tc_fence_after();
-      const int j0 = j * kKeys;
-      const bool edge = j0 + kKeys - 1 > a.start_pos + m0 || j0 + kKeys > p.n_keys;
+      const int j0 = first_key(j);
+      // a tile that every row sees whole needs no mask
+      const bool edge = j0 + kKeys - 1 > a.start_pos + m0 || j0 + kKeys > p.n_keys ||
+                        (j0 < window_start(a.start_pos + m0 + kRows - 1, a.window) && j0 + kKeys > a.keep_first);
       uint32_t x[4][32];
 #pragma unroll
       for (int c = 0; c < 4; ++c) tmem_ld32(ts + c * 32, x[c]);
@@ -236,7 +246,21 @@ mixer_tc_kernel(const __grid_constant__ CUtensorMap qamap, const __grid_constant
 #pragma unroll
           for (int i = 0; i < 32; ++i) {
             const int key = j0 + c * 32 + i;
-            if (key > limit || key >= p.n_keys) x[c][i] = 0xff800000u;  // -inf
+            if (key > limit || key >= p.n_keys || (key < row_lo && key >= a.keep_first)) x[c][i] = 0xff800000u;  // -inf
+          }
+      }
+      if (BIAS) {
+        // scores in the log2 domain with the distance taken off: slope * (i - (limit - j0)) for key j0 + i
+        const float base = slope * (float)(j0 - limit);
+        const unsigned long long sc2 = f2_packf(scale_log2e, scale_log2e), slope2 = f2_packf(slope, slope), base2 = f2_packf(base, base);
+#pragma unroll
+        for (int c = 0; c < 4; ++c)
+#pragma unroll
+          for (int i = 0; i < 32; i += 2) {
+            float t0, t1;
+            f2_unpack(f2_fma(f2_pack(x[c][i], x[c][i + 1]), sc2, f2_fma(f2_packf((float)(c * 32 + i), (float)(c * 32 + i + 1)), slope2, base2)), t0, t1);
+            x[c][i] = __float_as_uint(t0);
+            x[c][i + 1] = __float_as_uint(t1);
           }
       }
       float mx4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
@@ -245,7 +269,7 @@ mixer_tc_kernel(const __grid_constant__ CUtensorMap qamap, const __grid_constant
 #pragma unroll
         for (int i = 0; i < 32; i += 2)
           mx4[(i >> 1) & 3] = fmax3(mx4[(i >> 1) & 3], __uint_as_float(x[c][i]), __uint_as_float(x[c][i + 1]));
-      const float mx = fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3])) * scale_log2e;
+      const float mx = fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3])) * (BIAS ? 1.f : scale_log2e);
       if (__any_sync(kFullMask, mx > m_ref + kLazy)) {
         const float m_new = fmaxf(m_ref, mx);
         const float alpha = m_new == -INFINITY ? 1.f : fast_exp2(m_ref - m_new);
@@ -253,12 +277,12 @@ mixer_tc_kernel(const __grid_constant__ CUtensorMap qamap, const __grid_constant
           if (!mbar_wait_bounded(bar(O_FULL + e), (done - 1) & 1)) { ok = false; break; }
           tc_fence_after();
           rescale_row<D>(to, alpha);
-          l_run *= alpha;
         }
+        l_run *= alpha;
         m_ref = m_new;
       }
       const float mu = m_ref == -INFINITY ? 0.f : m_ref;
-      const unsigned long long scale2 = f2_packf(scale_log2e, scale_log2e), nmu2 = f2_packf(-mu, -mu);
+      const unsigned long long scale2 = f2_packf(BIAS ? 1.f : scale_log2e, BIAS ? 1.f : scale_log2e), nmu2 = f2_packf(-mu, -mu);
       unsigned long long ps2[4] = {0ull, 0ull, 0ull, 0ull};
 #pragma unroll
       for (int c = 0; c < 4; ++c) {
@@ -738,13 +762,13 @@ int set_smem(const void* fn, size_t smem, bool (&configured)[64]) {
   return L3CI_OK;
 }
 
-template <int KA, int KB, int VC>
+template <int KA, int KB, int VC, bool BIAS = false>
 int launch_one(const CUtensorMap (&m)[5], const TcMixParams& p, unsigned ctas, cudaStream_t stream) {
   constexpr size_t smem = 1024 + (size_t)((1 + kStages) * (KA + KB) + kStages * VC) * kBox + 15 * 8 + 4 * kRows * 4 + 16;
   static_assert(smem <= (227 << 10), "shared memory");
   static bool configured[64] = {false};
-  if (int st = set_smem(reinterpret_cast<const void*>(mixer_tc_kernel<KA, KB, VC>), smem, configured)) return st;
-  mixer_tc_kernel<KA, KB, VC><<<ctas, kOneThreads, smem, stream>>>(m[0], m[1], m[2], m[3], m[4], p);
+  if (int st = set_smem(reinterpret_cast<const void*>(mixer_tc_kernel<KA, KB, VC, BIAS>), smem, configured)) return st;
+  mixer_tc_kernel<KA, KB, VC, BIAS><<<ctas, kOneThreads, smem, stream>>>(m[0], m[1], m[2], m[3], m[4], p);
   L3CI_CHECK_LAUNCH("mixer_tc_kernel");
   return L3CI_OK;
 }
@@ -765,6 +789,7 @@ int launch_maps(const CUtensorMap& q0, const CUtensorMap& q1, const CUtensorMap&
 bool mixer_tc_applies(const l3ci_mixer_attn_args* a) {
   if (a->dtype != L3CI_BF16 || a->start_pos < 0 || a->start_pos + a->T > a->n_keys || a->Dv > 128 || a->Dv % 8 || a->Da % 8 || a->Db % 8)
     return false;
+  if (a->maps == 1 && a->bias_range > 0.f && a->Db) return false;
   if (a->maps == 2 ? a->Da > 64 : a->Da > 128 || a->Db > 64 || a->softcap > 0.f || a->temp_every > 0.f || !(a->scale > 0.f)) return false;
   if ((long long)a->B * a->H * ((a->T + kRows - 1) / kRows) > 0x7fffffffLL) return false;
   // rows the copy engine can address: positive strides of whole 16-byte vectors (an axis of extent 1 may have any)
@@ -820,6 +845,10 @@ int mixer_tc_launch(const l3ci_mixer_attn_args* a) {
   if (kb) {
     if (ka == 1) return vc == 1 ? launch_one<1, 1, 1>(m, p, ctas, stream) : launch_one<1, 1, 2>(m, p, ctas, stream);
     return vc == 1 ? launch_one<2, 1, 1>(m, p, ctas, stream) : launch_one<2, 1, 2>(m, p, ctas, stream);
+  }
+  if (a->bias_range > 0.f) {
+    if (ka == 1) return vc == 1 ? launch_one<1, 0, 1, true>(m, p, ctas, stream) : launch_one<1, 0, 2, true>(m, p, ctas, stream);
+    return vc == 1 ? launch_one<2, 0, 1, true>(m, p, ctas, stream) : launch_one<2, 0, 2, true>(m, p, ctas, stream);
   }
   if (ka == 1) return vc == 1 ? launch_one<1, 0, 1>(m, p, ctas, stream) : launch_one<1, 0, 2>(m, p, ctas, stream);
   return vc == 1 ? launch_one<2, 0, 1>(m, p, ctas, stream) : launch_one<2, 0, 2>(m, p, ctas, stream);

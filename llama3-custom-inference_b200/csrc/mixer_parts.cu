@@ -1,6 +1,6 @@
 // The memory-bound steps around the mixers of a decoder with a 32-bit residual stream: residual add + dynamic-tanh
-// norm (with the embedding lookup as its first form), exact gelu, and the passes that turn a fused projection row
-// into queries and cache rows.  Storage is bf16 or fp32 (template), arithmetic fp32.
+// norm (with the embedding lookup as its first form), activations, the passes that turn a fused projection row into
+// queries and cache rows, and the mixes of a token with the one before it.  Storage is bf16 or fp32 (template), arithmetic fp32.
 #include <cuda_bf16.h>
 #include <cuda_runtime.h>
 
@@ -52,8 +52,10 @@ add_dyn_tanh_kernel(const S* __restrict__ y, const long long* __restrict__ token
   }
 }
 
-template <typename S, int VEC>
-__global__ void __launch_bounds__(256) gelu_kernel(const S* __restrict__ z, S* __restrict__ out, long long n) {
+enum { kGelu = 0, kTanh = 1 };
+
+template <typename S, int VEC, int KIND>
+__global__ void __launch_bounds__(256) activation_kernel(const S* __restrict__ z, S* __restrict__ out, long long n) {
   pdl_wait();
   pdl_launch_dependents();
   const long long i0 = ((long long)blockIdx.x * 256 + threadIdx.x) * VEC;
@@ -61,8 +63,119 @@ __global__ void __launch_bounds__(256) gelu_kernel(const S* __restrict__ z, S* _
   float v[VEC];
   load_vec<S, VEC>(z + i0, v);
 #pragma unroll
-  for (int i = 0; i < VEC; ++i) v[i] = 0.5f * v[i] * (1.f + erff(v[i] * 0.70710678118654752f));
+  for (int i = 0; i < VEC; ++i) v[i] = KIND == kTanh ? tanhf(v[i]) : 0.5f * v[i] * (1.f + erff(v[i] * 0.70710678118654752f));
   store_vec<S, VEC>(out + i0, v);
+}
+
+// ---- gated feed-forward activation of rows [gate | up] -----------------------------------------------------------
+template <typename S, int VEC>
+__global__ void __launch_bounds__(256)
+gated_act_kernel(const S* __restrict__ gu, S* __restrict__ out, long long units, int per_row, float limit, float alpha) {
+  pdl_wait();
+  pdl_launch_dependents();
+  const long long id = (long long)blockIdx.x * 256 + threadIdx.x;
+  if (id >= units) return;
+  const long long row = units <= 0xffffffffLL ? (unsigned)id / (unsigned)per_row : id / per_row;
+  const int c = (int)(id - row * per_row) * VEC, ff = per_row * VEC;
+  float g[VEC], u[VEC];
+  load_vec<S, VEC>(gu + row * 2 * ff + c, g);
+  load_vec<S, VEC>(gu + row * 2 * ff + ff + c, u);
+#pragma unroll
+  for (int i = 0; i < VEC; ++i) g[i] = gated_activation(g[i], u[i], limit, alpha);
+  store_vec<S, VEC>(out + row * ff + c, g);
+}
+
+// ---- whole-row RMS norm of q and k, k and v into the caches ------------------------------------------------------
+struct QkNormRow {
+  long long stride, k_sb, k_st, v_sb, v_st, cache_len;
+  int q_width, k_width, v_width, T;
+  float eps;
+};
+
+template <typename S, int VEC>
+__global__ void __launch_bounds__(256)
+qk_norm_cache_kernel(S* __restrict__ qkv, const float* __restrict__ qw, const float* __restrict__ kw, S* __restrict__ ck,
+                     S* __restrict__ cv, const int* __restrict__ positions, const QkNormRow p) {
+  __shared__ float red[2][8];
+  pdl_wait();
+  pdl_launch_dependents();
+  const long long row = blockIdx.x;
+  const int b = (int)(row / p.T), t = (int)(row % p.T), tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, warps = blockDim.x / kWarp;
+  const long long pos = (long long)positions[b] + t;
+  S* r = qkv + row * p.stride;
+  const int qk = p.q_width + p.k_width, step = blockDim.x * VEC;
+  float ss[2] = {0.f, 0.f};
+  for (int c = tid * VEC; c < qk; c += step) {
+    float f[VEC];
+    load_vec<S, VEC>(r + c, f);
+    const int part = c < p.q_width ? 0 : 1;
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) {
+      if (part == 0) ss[0] = fmaf(f[i], f[i], ss[0]);
+      else ss[1] = fmaf(f[i], f[i], ss[1]);
+    }
+  }
+#pragma unroll
+  for (int i = 0; i < 2; ++i) ss[i] = group_sum<kWarp>(ss[i]);
+  if (lane == 0) {
+    red[0][warp] = ss[0];
+    red[1][warp] = ss[1];
+  }
+  __syncthreads();
+#pragma unroll
+  for (int i = 0; i < 2; ++i) ss[i] = group_sum<8>(lane % 8 < warps ? red[i][lane % 8] : 0.f);
+  const float iq = 1.f / sqrtf(ss[0] / (float)p.q_width + p.eps), ik = 1.f / sqrtf(ss[1] / (float)p.k_width + p.eps);
+  const bool cached = pos >= 0 && pos < p.cache_len;
+  S* kr = ck + b * p.k_sb + pos * p.k_st;
+  S* vr = cv + b * p.v_sb + pos * p.v_st;
+  for (int c = tid * VEC; c < qk + p.v_width; c += step) {
+    float f[VEC], w[VEC];
+    load_vec<S, VEC>(r + c, f);
+    if (c < qk) {
+      const bool is_q = c < p.q_width;
+      load_vec<float, VEC>(is_q ? qw + c : kw + (c - p.q_width), w);
+#pragma unroll
+      for (int i = 0; i < VEC; ++i) f[i] = f[i] * (is_q ? iq : ik) * w[i];
+      if (is_q) store_vec<S, VEC>(r + c, f);
+      else if (cached) store_vec<S, VEC>(kr + (c - p.q_width), f);
+    } else if (cached) {
+      store_vec<S, VEC>(vr + (c - qk), f);
+    }
+  }
+}
+
+// ---- token shift: n mixes of a row with the one before it ----------------------------------------------------------
+template <typename S, int VEC>
+__global__ void __launch_bounds__(256)
+token_shift_kernel(const S* __restrict__ h, const float* __restrict__ mu, S* __restrict__ last, long long last_sb,
+                   const int* __restrict__ positions, S* __restrict__ out, int n_mix, int T, long long rows, int width) {
+  pdl_wait();
+  pdl_launch_dependents();
+  const long long row = blockIdx.x;
+  const int b = (int)(row / T), t = (int)(row % T);
+  const bool fresh = positions[b] == 0;
+  S* carried = last + b * last_sb;
+  for (int c = threadIdx.x * VEC; c < width; c += blockDim.x * VEC) {
+    float x[VEC], d[VEC] = {};
+    load_vec<S, VEC>(h + row * width + c, x);
+    if (t > 0) {
+      load_vec<S, VEC>(h + (row - 1) * width + c, d);
+    } else {
+      if (!fresh) load_vec<S, VEC>(carried + c, d);
+      float end[VEC];                                       // the thread that has read the old value writes the new one
+      load_vec<S, VEC>(h + (row + T - 1) * width + c, end);
+      store_vec<S, VEC>(carried + c, end);
+    }
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) d[i] -= x[i];
+    for (int s = 0; s < n_mix; ++s) {
+      float m[VEC];
+      load_vec<float, VEC>(mu + (long long)s * width + c, m);
+#pragma unroll
+      for (int i = 0; i < VEC; ++i) m[i] = fmaf(d[i], m[i], x[i]);
+      store_vec<S, VEC>(out + ((long long)s * rows + row) * width + c, m);
+    }
+  }
 }
 
 // ---- latent attention: query rotation in place, latent norm, key rotation, cache row ---------------------------
@@ -331,17 +444,26 @@ int add_dyn_tanh_typed(const void* y, const int64_t* tokens, const void* table, 
   return v4 ? go(add_dyn_tanh_kernel<S, 4>) : go(add_dyn_tanh_kernel<S, 1>);
 }
 
-template <typename S>
-int gelu_typed(const void* z, void* out, int64_t n, cudaStream_t stream) {
+template <typename S, int KIND>
+int activation_typed(const void* z, void* out, int64_t n, cudaStream_t stream) {
   constexpr int kVec = 16 / sizeof(S);
   const bool v = n % kVec == 0 && vec_ok<S>(z, kVec) && vec_ok<S>(out, kVec);
   const long long units = v ? n / kVec : n, ctas = (units + 255) / 256;
-  if (ctas > 0x7fffffffLL) return fail(L3CI_ERR_INVALID, "gelu: tensor too large");
+  if (ctas > 0x7fffffffLL) return fail(L3CI_ERR_INVALID, "activation: tensor too large");
   auto go = [&](auto kernel) -> int {
-    L3CI_LAUNCH("gelu_kernel", kernel, dim3((unsigned)ctas), dim3(256), 0, stream, static_cast<const S*>(z), static_cast<S*>(out), (long long)n);
+    L3CI_LAUNCH("activation_kernel", kernel, dim3((unsigned)ctas), dim3(256), 0, stream, static_cast<const S*>(z), static_cast<S*>(out), (long long)n);
     return L3CI_OK;
   };
-  return v ? go(gelu_kernel<S, kVec>) : go(gelu_kernel<S, 1>);
+  return v ? go(activation_kernel<S, kVec, KIND>) : go(activation_kernel<S, 1, KIND>);
+}
+
+template <int KIND>
+int activation(const char* name, const void* z, void* out, int64_t n, int32_t dtype, cudaStream_t stream) {
+  clear_error();
+  if (n < 0 || bad_dtype(dtype)) return fail(L3CI_ERR_INVALID, "%s: n=%lld dtype=%d", name, (long long)n, dtype);
+  if (n == 0) return L3CI_OK;
+  if (!z || !out) return fail(L3CI_ERR_INVALID, "%s: null pointer", name);
+  return dtype == L3CI_BF16 ? activation_typed<__nv_bfloat16, KIND>(z, out, n, stream) : activation_typed<float, KIND>(z, out, n, stream);
 }
 
 }  // namespace
@@ -367,14 +489,102 @@ int l3ci_add_dyn_tanh(const void* y, const int64_t* tokens, const void* table, i
                             : add_dyn_tanh_typed<float>(y, tokens, table, vocab, x, weight, bias, alpha, out, rows, width, s);
 }
 
-int l3ci_gelu(const void* z, void* out, int64_t n, int32_t dtype, l3ci_stream_t stream_) {
+int l3ci_gelu(const void* z, void* out, int64_t n, int32_t dtype, l3ci_stream_t stream) {
+  return l3ci::activation<l3ci::kGelu>("gelu", z, out, n, dtype, reinterpret_cast<cudaStream_t>(stream));
+}
+
+int l3ci_tanh(const void* z, void* out, int64_t n, int32_t dtype, l3ci_stream_t stream) {
+  return l3ci::activation<l3ci::kTanh>("tanh", z, out, n, dtype, reinterpret_cast<cudaStream_t>(stream));
+}
+
+int l3ci_gated_act(const void* gu, void* out, int64_t rows, int64_t ff, float limit, float alpha, int32_t dtype, l3ci_stream_t stream_) {
   using namespace l3ci;
   clear_error();
-  if (n < 0 || bad_dtype(dtype)) return fail(L3CI_ERR_INVALID, "gelu: n=%lld dtype=%d", (long long)n, dtype);
-  if (n == 0) return L3CI_OK;
-  if (!z || !out) return fail(L3CI_ERR_INVALID, "gelu: null pointer");
+  if (rows < 0 || ff <= 0 || ff > 0x3fffffffLL || bad_dtype(dtype) || !(limit >= 0.f))
+    return fail(L3CI_ERR_INVALID, "gated_act: rows=%lld ff=%lld dtype=%d", (long long)rows, (long long)ff, dtype);
+  if (rows == 0) return L3CI_OK;
+  if (!gu || !out) return fail(L3CI_ERR_INVALID, "gated_act: null pointer");
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream_);
-  return dtype == L3CI_BF16 ? gelu_typed<__nv_bfloat16>(z, out, n, s) : gelu_typed<float>(z, out, n, s);
+  auto typed = [&](auto zero) -> int {
+    using S = decltype(zero);
+    constexpr int kVec = 16 / sizeof(S);
+    const bool v = ff % kVec == 0 && aligned16(gu) && aligned16(out);
+    const long long units = rows * (v ? ff / kVec : ff), ctas = (units + 255) / 256;
+    if (ctas > 0x7fffffffLL) return fail(L3CI_ERR_INVALID, "gated_act: too much");
+    auto go = [&](auto kernel) -> int {
+      L3CI_LAUNCH("gated_act_kernel", kernel, dim3((unsigned)ctas), dim3(256), 0, s, static_cast<const S*>(gu), static_cast<S*>(out), units,
+                  (int)(units / rows), limit, alpha);
+      return L3CI_OK;
+    };
+    return v ? go(gated_act_kernel<S, kVec>) : go(gated_act_kernel<S, 1>);
+  };
+  return dtype == L3CI_BF16 ? typed(__nv_bfloat16{}) : typed(float{});
+}
+
+int l3ci_qk_norm_cache(void* qkv, int64_t stride, int64_t q_width, int64_t k_width, int64_t v_width, const float* q_norm,
+                       const float* k_norm, float eps, void* cache_k, int64_t k_sb, int64_t k_st, void* cache_v, int64_t v_sb,
+                       int64_t v_st, int64_t cache_len, const int32_t* positions, int32_t B, int32_t T, int32_t dtype,
+                       l3ci_stream_t stream_) {
+  using namespace l3ci;
+  clear_error();
+  if (B < 0 || T < 0 || q_width <= 0 || k_width <= 0 || v_width <= 0 || q_width + k_width + v_width > 0x3fffffffLL ||
+      stride < q_width + k_width + v_width || bad_dtype(dtype))
+    return fail(L3CI_ERR_INVALID, "qk_norm_cache: B=%d T=%d widths %lld %lld %lld", B, T, (long long)q_width, (long long)k_width, (long long)v_width);
+  if (B == 0 || T == 0) return L3CI_OK;
+  if (!qkv || !q_norm || !k_norm || !cache_k || !cache_v || !positions) return fail(L3CI_ERR_INVALID, "qk_norm_cache: null pointer");
+  const long long rows = (long long)B * T;
+  if (rows > 0x7fffffffLL) return fail(L3CI_ERR_INVALID, "qk_norm_cache: too many rows");
+  const QkNormRow p{stride, k_sb, k_st, v_sb, v_st, cache_len, (int)q_width, (int)k_width, (int)v_width, T, eps};
+  cudaStream_t s = reinterpret_cast<cudaStream_t>(stream_);
+  auto typed = [&](auto zero) -> int {
+    using S = decltype(zero);
+    constexpr int kVec = 16 / sizeof(S);
+    const int64_t all = stride | q_width | k_width | v_width | k_sb | k_st | v_sb | v_st;
+    const bool v = all % kVec == 0 && aligned16(qkv) && aligned16(cache_k) && aligned16(cache_v) && aligned16(q_norm) && aligned16(k_norm);
+    const long long units = (q_width + k_width + v_width) / (v ? kVec : 1);
+    int threads = 32;
+    while (threads < 256 && threads < units) threads *= 2;
+    auto go = [&](auto kernel) -> int {
+      L3CI_LAUNCH("qk_norm_cache_kernel", kernel, dim3((unsigned)rows), dim3(threads), 0, s, static_cast<S*>(qkv), q_norm, k_norm,
+                  static_cast<S*>(cache_k), static_cast<S*>(cache_v), positions, p);
+      return L3CI_OK;
+    };
+    if constexpr (sizeof(S) == 4) {
+      return v ? go(qk_norm_cache_kernel<S, 4>) : go(qk_norm_cache_kernel<S, 1>);
+    } else {
+      // (weights are read in as many elements as the row: 32 bytes, two accesses)
+      return v ? go(qk_norm_cache_kernel<S, 8>) : go(qk_norm_cache_kernel<S, 1>);
+    }
+  };
+  return dtype == L3CI_BF16 ? typed(__nv_bfloat16{}) : typed(float{});
+}
+
+int l3ci_token_shift(const void* h, const float* mu, void* last, int64_t last_sb, const int32_t* positions, void* out, int32_t n_mix,
+                     int32_t B, int32_t T, int64_t width, int32_t dtype, l3ci_stream_t stream_) {
+  using namespace l3ci;
+  clear_error();
+  if (B < 0 || T < 0 || n_mix <= 0 || width <= 0 || width > 0x3fffffffLL || bad_dtype(dtype) || (B > 1 && last_sb < width))
+    return fail(L3CI_ERR_INVALID, "token_shift: B=%d T=%d n_mix=%d width=%lld", B, T, n_mix, (long long)width);
+  if (B == 0 || T == 0) return L3CI_OK;
+  if (!h || !mu || !last || !positions || !out) return fail(L3CI_ERR_INVALID, "token_shift: null pointer");
+  const long long rows = (long long)B * T;
+  if (rows > 0x7fffffffLL) return fail(L3CI_ERR_INVALID, "token_shift: too many rows");
+  cudaStream_t s = reinterpret_cast<cudaStream_t>(stream_);
+  auto typed = [&](auto zero) -> int {
+    using S = decltype(zero);
+    constexpr int kVec = 16 / sizeof(S);
+    const bool v = (width | last_sb) % kVec == 0 && aligned16(h) && aligned16(mu) && aligned16(last) && aligned16(out);
+    const long long units = width / (v ? kVec : 1);
+    int threads = 32;
+    while (threads < 256 && threads < units) threads *= 2;
+    auto go = [&](auto kernel) -> int {
+      L3CI_LAUNCH("token_shift_kernel", kernel, dim3((unsigned)rows), dim3(threads), 0, s, static_cast<const S*>(h), mu, static_cast<S*>(last),
+                  (long long)last_sb, positions, static_cast<S*>(out), n_mix, T, rows, (int)width);
+      return L3CI_OK;
+    };
+    return v ? go(token_shift_kernel<S, kVec>) : go(token_shift_kernel<S, 1>);
+  };
+  return dtype == L3CI_BF16 ? typed(__nv_bfloat16{}) : typed(float{});
 }
 
 int l3ci_latent_cache(void* qd, int64_t qd_stride, const float* table, int64_t table_rows, const float* norm_weight, float eps,

@@ -17,6 +17,17 @@ __device__ __forceinline__ float from_f32<float>(float v) { return v; }
 template <>
 __device__ __forceinline__ __nv_bfloat16 from_f32<__nv_bfloat16>(float v) { return __float2bfloat16_rn(v); }
 
+// A gate z with its partner u: silu(z) u, or, with a limit, z' sigmoid(alpha z') (u' + 1) of the clamped z' = min(z, limit) and
+// u' = clamp(u, -limit, limit).
+__device__ __forceinline__ float gated_activation(float z, float u, float limit, float alpha) {
+  if (limit > 0.f) {
+    z = fminf(z, limit);
+    u = fminf(fmaxf(u, -limit), limit) + 1.f;
+    return z / (1.f + expf(-alpha * z)) * u;
+  }
+  return z / (1.f + expf(-z)) * u;
+}
+
 template <int BYTES>
 struct Raw;
 template <>
@@ -27,6 +38,9 @@ template <>
 struct Raw<8> { using type = uint2; };
 template <>
 struct Raw<16> { using type = uint4; };
+struct alignas(16) Raw32 { uint4 lo, hi; };
+template <>
+struct Raw<32> { using type = Raw32; };   // two accesses
 
 template <typename S, int VEC>
 __device__ __forceinline__ void load_vec(const S* p, float (&f)[VEC]) {

@@ -11,7 +11,7 @@ from typing import Callable
 
 import torch
 
-from . import build, checkpoint, decode_loop, nibelorn
+from . import build, checkpoint, decode_loop, nibelorn, rupotar
 
 
 @dataclass(frozen=True)
@@ -30,6 +30,9 @@ ARCHITECTURES = {
     "Nibelorn": Architecture(
         read_config=nibelorn.config_from_json, map_weights=lambda tensors, cfg: tensors,
         decoder=nibelorn.NibelornDecoder, libraries=("mixers",), dtypes=(torch.bfloat16, torch.float32)),
+    "Rupotar": Architecture(
+        read_config=rupotar.config_from_json, map_weights=lambda tensors, cfg: tensors,
+        decoder=rupotar.RupotarDecoder, libraries=("mixers",), dtypes=(torch.bfloat16, torch.float32)),
 }
 
 
