@@ -178,11 +178,17 @@ def gated_act(gu, limit: float = 0.0, alpha: float = 1.702):
     return out
 
 
+def _row_stride(t) -> int:
+    """Elements between consecutive rows of t [B, T, ...], (b, t) pairs counted as one axis."""
+    B, T = t.shape[:2]
+    assert t.stride(-1) == 1 and (B == 1 or T == 1 or t.stride(0) == T * t.stride(1))
+    return t.stride(1) if T > 1 else t.stride(0) if B > 1 else t[0, 0].numel()
+
+
 def _residual(a: ResidualNormArgs, x, out):
     a.x, a.rows, a.width = x.data_ptr(), x.numel() // x.shape[-1], x.shape[-1]
     if out is not None:
-        assert out.stride(-1) == 1 and (out.dim() < 3 or out.stride(0) == out.shape[1] * out.stride(1))
-        a.out, a.out_stride = out.data_ptr(), out.stride(-2)
+        a.out, a.out_stride = out.data_ptr(), _row_stride(out if out.dim() > 2 else out[None])
     a.stream = _stream(x)
     with _on(x):
         _check(load().l3ci_residual_norm(C.byref(a)), "l3ci_residual_norm")
@@ -206,8 +212,8 @@ def embed_residual(tokens, table, scale: float, freqs, positions, x0=None, norm=
         assert freqs.dtype == torch.float64 and freqs.numel() == (E + 1) // 2
         a.freqs = freqs.data_ptr()
     if x0 is not None:
-        assert x0.dtype == table.dtype and x0.stride(-1) == 1 and x0.stride(0) == T * x0.stride(1)
-        a.x0, a.x0_stride = x0.data_ptr(), x0.stride(-2)
+        assert x0.dtype == table.dtype
+        a.x0, a.x0_stride = x0.data_ptr(), _row_stride(x0)
     if norm is not None:
         a.pre_w, a.pre_b = norm[0].data_ptr(), norm[1].data_ptr()
     _residual(a, x, out)
@@ -271,15 +277,14 @@ def delta_inputs(p, b, a_proj, conv, a_log, dt_bias, tail, positions, H: int, G:
     _cuda(p, b, a_proj, tail, positions)
     B, T, _ = p.shape
     dev, f32 = p.device, torch.float32
-    for t in (p, b, a_proj):
-        assert t.stride(-1) == 1 and t.stride(0) == T * t.stride(1) and t.dtype == p.dtype
+    assert b.dtype == a_proj.dtype == p.dtype
     assert conv.is_contiguous() and tail[0].is_contiguous() and tail.dtype == p.dtype
     qk, beta = torch.empty(B, T, 2, G, D, dtype=f32, device=dev), torch.empty(B, T, H, dtype=f32, device=dev)
     decay, v = torch.empty(B, T, H, D, dtype=f32, device=dev), torch.empty(B, T, H, V, dtype=p.dtype, device=dev)
     a = DeltaInputsArgs(p=p.data_ptr(), b=b.data_ptr(), a=a_proj.data_ptr(), conv=conv.data_ptr(), a_log=a_log.data_ptr(),
                         dt_bias=dt_bias.data_ptr(), tail=tail.data_ptr(), positions=positions.data_ptr(), qk_out=qk.data_ptr(),
-                        beta_out=beta.data_ptr(), decay_out=decay.data_ptr(), v_out=v.data_ptr(), p_st=p.stride(1), b_st=b.stride(1),
-                        a_st=a_proj.stride(1), tail_sb=tail.stride(0), B=B, T=T, H=H, G=G, D=D, V=V, taps=conv.shape[0],
+                        beta_out=beta.data_ptr(), decay_out=decay.data_ptr(), v_out=v.data_ptr(), p_st=_row_stride(p), b_st=_row_stride(b),
+                        a_st=_row_stride(a_proj), tail_sb=tail.stride(0), B=B, T=T, H=H, G=G, D=D, V=V, taps=conv.shape[0],
                         dtype=DTYPE_CODES[p.dtype], unit_eps=unit_eps, stream=_stream(p))
     with _on(p):
         _check(load().l3ci_delta_inputs(C.byref(a)), "l3ci_delta_inputs")
@@ -295,13 +300,11 @@ def recurrent_scan(q, k, v, g, state, positions, norm, gate, *, act: int, eps: f
     B, T, H, V = v.shape
     G, D = q.shape[2:]
     out = torch.empty(B, T, H, V, dtype=v.dtype, device=v.device)
-    for t in (q, k, g, v, gate):
-        assert t.stride(-1) == 1 and t.stride(0) == T * t.stride(1)
-    assert k.stride() == q.stride() and gate.dtype == v.dtype and state.dtype == torch.float32 and state[0].is_contiguous()
+    assert _row_stride(k) == _row_stride(q) and k.stride(2) == q.stride(2) and gate.dtype == v.dtype and state.dtype == torch.float32 and state[0].is_contiguous()
     assert q.dtype == k.dtype == g.dtype == (torch.float32 if beta is not None else v.dtype) and norm.is_contiguous()
     a = RecurrentScanArgs(q=q.data_ptr(), k=k.data_ptr(), v=v.data_ptr(), g=g.data_ptr(), norm=norm.data_ptr(), gate=gate.data_ptr(),
-                          state=state.data_ptr(), out=out.data_ptr(), positions=positions.data_ptr(), qk_st=q.stride(1), qk_sh=q.stride(2),
-                          v_st=v.stride(1), v_sh=v.stride(2), g_st=g.stride(1), g_sh=g.stride(2), gate_st=gate.stride(1),
+                          state=state.data_ptr(), out=out.data_ptr(), positions=positions.data_ptr(), qk_st=_row_stride(q), qk_sh=q.stride(2),
+                          v_st=_row_stride(v), v_sh=v.stride(2), g_st=_row_stride(g), g_sh=g.stride(2), gate_st=_row_stride(gate),
                           gate_sh=gate.stride(2), out_st=H * V, out_sh=V, norm_sh=V if norm.dim() == 2 else 0,
                           state_sb=state.stride(0), kind=0 if beta is not None else 1, B=B, T=T, H=H, G=G, D=D, V=V, act=act,
                           taps=taps, dtype=DTYPE_CODES[v.dtype], eps=eps, stream=_stream(v))
@@ -312,8 +315,8 @@ def recurrent_scan(q, k, v, g, state, positions, norm, gate, *, act: int, eps: f
     if status is not None:
         a.status = status.data_ptr()
     if tail is not None:
-        assert conv_in.stride(-1) == 1 and conv_in.stride(0) == T * conv_in.stride(1) and tail[0].is_contiguous()
-        a.conv_in, a.conv_st, a.tail, a.tail_sb = conv_in.data_ptr(), conv_in.stride(1), tail.data_ptr(), tail.stride(0)
+        assert tail[0].is_contiguous() and conv_in.dtype == tail.dtype == v.dtype
+        a.conv_in, a.conv_st, a.tail, a.tail_sb = conv_in.data_ptr(), _row_stride(conv_in), tail.data_ptr(), tail.stride(0)
     with _on(v):
         _check(load().l3ci_recurrent_scan(C.byref(a)), "l3ci_recurrent_scan")
     return out.view(B, T, H * V)

@@ -127,7 +127,7 @@ def test_mixer_header_and_binding_agree(pkg):
     names = re.findall(r"\b(\w+)(?=[,;])", text[text.index("typedef struct l3ci_mixer_attn_args"):text.index("} l3ci_mixer_attn_args")].replace("*", " "))
     fields = [n.rstrip("_") for n, _ in pkg.mixers.AttnArgs._fields_]
     assert [n for n in names if n in fields] == fields   # same members, same order
-    assert C.sizeof(pkg.mixers.AttnArgs) == 11 * 8 + 20 * 8 + 12 * 4 + 7 * 4 + 4 + 8
+    assert C.sizeof(pkg.mixers.AttnArgs) == 11 * 8 + 20 * 8 + 15 * 4 + 8 * 4 + 4 + 8
 
 
 def test_mixer_arguments_are_validated_before_cuda(pkg):
