@@ -1,7 +1,7 @@
 #!/usr/bin/env python
 """Benchmark of the decode hot path on B200.
 
-    python bench.py [--gpus N] [--steps K] [--warmup W] [--workload c2|c1|c3|rmsnorm|rope|c5|prefill|nibelorn]
+    python bench.py [--gpus N] [--steps K] [--warmup W] [--workload c2|c1|c3|rmsnorm|rope|c5|prefill|nibelorn|rupotar]
                     [--impl ours|reference]
 
 One "step" is one pass of the hot path over one batch of synthetic input: for the default workload (C2) one
@@ -31,6 +31,9 @@ Printed JSON line (rank 0):
   --workload nibelorn
                  the Nibelorn decoder at the layer sizes of a 1B model beside the Llama-3 decoder of equal size: prefill and
                  decode tokens/s at a few batches, and every mixer kernel's roofline beside its Llama-3 counterpart's
+  --workload rupotar
+                 the same for the Rupotar decoder (windowed attention, two recurrences, experts, looped layers) beside the
+                 Nibelorn decoder of equal width, depth and active feed-forward size
   comparators    torch's SDPA on the same GPU tensors; and, at N = 1, the reference's own CUDA kernels rebuilt
                  for sm_100 (oracle/_ref, when present), timed beside this library's calls
 
@@ -268,7 +271,7 @@ def main():
     ap.add_argument("--gpus", type=int, default=1)
     ap.add_argument("--steps", type=int, default=2000)
     ap.add_argument("--warmup", type=int, default=100)
-    ap.add_argument("--workload", default=None, choices=["c1", "c2", "c3", "rmsnorm", "rope", "c5", "prefill", "nibelorn"],
+    ap.add_argument("--workload", default=None, choices=["c1", "c2", "c3", "rmsnorm", "rope", "c5", "prefill", "nibelorn", "rupotar"],
                     help="default: c2 as the headline plus the sub-records of the other configurations")
     ap.add_argument("--gen-len", type=int, default=2048, help="c5: tokens generated per sequence")
     ap.add_argument("--batch", type=int, default=64, help="c5: sequences per GPU")
@@ -318,6 +321,8 @@ def main():
         line = bench_end_to_end(args, ext, pkg, dev, rank, world)
     elif args.workload == "nibelorn":
         line = bench_nibelorn(args, ext, pkg, dev, rank, world)
+    elif args.workload == "rupotar":
+        line = bench_rupotar(args, ext, pkg, dev, rank, world)
     elif args.workload == "prefill":
         line = bench_prefill(args, ext, pkg, dev, rank, world)
     elif args.workload in ("rmsnorm", "rope"):
@@ -1042,22 +1047,20 @@ def bench_end_to_end(args, ext, pkg, dev, rank, world):
     return line
 
 
-def bench_nibelorn(args, ext, pkg, dev, rank, world):
-    """The Nibelorn decoder (random weights) at a 1B model's layer sizes: width 2048, 16 layers, latent and differential
-    attention in turn, feed-forward 8192, vocabulary 128256, beside the Llama-3 decoder of the same width, depth,
-    feed-forward size and vocabulary.  Value: decode tokens/s at batch 64 behind 1024-token prompts, by CUDA events
-    around the replayed decode steps of a generation (prefill and graph capture are not in it; prefill is timed alone)."""
-    nb, dl = pkg.nibelorn, pkg.decode_loop
+def nibelorn_layers(nb):
     latent = nb.LatentAttention(heads=16, dim=128, rot_dim=64, vdim=128, kv_rank=512, scale=192 ** -0.5, rot_base=10000.0)
     differential = nb.DifferentialAttention(heads=16, kv_heads=4, dim=64, vdim=128, scale=0.125, diff=0.5, softcap=50.0, temp_coef=0.3,
                                             temp_every=256.0)
-    cfg = nb.NibelornConfig(128256, 2048, 1e-5, tuple(nb.Layer((latent, differential)[i % 2], 8192, i) for i in range(16)))
-    llama = dl.DecoderConfig()
+    return latent, differential, nb.NibelornConfig(128256, 2048, 1e-5, tuple(nb.Layer((latent, differential)[i % 2], 8192, i) for i in range(16)))
+
+
+def bench_decoders(decoders, ext, dev, rank, world):
+    """Prefill and decode of several decoders, name -> (class, configuration, weights()), at a few batches: decode by CUDA events
+    around the replayed steps of a generation (prefill and graph capture are not in it), prefill alone, and the first
+    decoder's end-to-end call at the largest batch."""
     short, long = 17, 129
     shapes = ((64, 1024), (8, 4096), (1, 8192))
-    weights = {"nibelorn": lambda: nb.init_weights(cfg, 42 + rank, dev),
-               "llama3": lambda: {k: v.to(dev) for k, v in dl.init_weights(llama, 42 + rank).items()}}
-    decoders = {"nibelorn": (nb.NibelornDecoder, cfg), "llama3": (dl.Llama3Decoder, llama)}
+    head = next(iter(decoders))
 
     def timed(fn, repeats=3):
         times = []
@@ -1074,14 +1077,14 @@ def bench_nibelorn(args, ext, pkg, dev, rank, world):
     sampler = ClockSampler(dev.index or 0)
     sampler.start()
     models, e2e = {}, None
-    for name, (decoder, config) in decoders.items():
-        w = weights[name]()
+    for name, (decoder, config, make_weights) in decoders.items():
+        w = make_weights()
         models[name] = {}
         for B, P in shapes:
             model = decoder(ext, config, dev, B, P + long, weights=dict(w))
             prompts = torch.randint(0, 128256, (B, P), generator=torch.Generator().manual_seed(7 + rank)).to(dev)
             model.generate(prompts, short)
-            if (name, B) == ("nibelorn", 64):
+            if (name, B) == (head, 64):
                 sampler.mark("t0")
             prefill = timed(lambda: model.generate(prompts, 1))
             steps = []
@@ -1092,7 +1095,7 @@ def bench_nibelorn(args, ext, pkg, dev, rank, world):
                 torch.cuda.synchronize()
                 steps.append(timing["events"][0].elapsed_time(timing["events"][1]) / timing["steps"])
             step = max_over_ranks(sorted(steps)[1], world, dev)
-            if (name, B) == ("nibelorn", 64):
+            if (name, B) == (head, 64):
                 sampler.mark("t1")
                 host, back = prompts.cpu().pin_memory(), torch.empty(B, long, dtype=torch.int64).pin_memory()
 
@@ -1108,35 +1111,85 @@ def bench_nibelorn(args, ext, pkg, dev, rank, world):
             del model
             torch.cuda.empty_cache()
         del w
+        torch.cuda.empty_cache()
     sampler.stop()
-    head = models["nibelorn"]["B=64 prompt=1024"]
+    value = models[head]["B=64 prompt=1024"]
+    return {"value": value["decode_tokens_per_s"], "unit": "tokens/s", "n_gpus": world, "steps": long - 2, "warmup": short,
+            "ms_per_step": value["decode_ms_per_step"], "higher_is_better": True, "scaling": "weak", "vs_baseline": None, "dtype": "bf16",
+            "data": "synthetic", "models": models, "e2e": e2e, "clocks": sampler.summary()}
+
+
+def bench_nibelorn(args, ext, pkg, dev, rank, world):
+    """The Nibelorn decoder (random weights) at a 1B model's layer sizes: width 2048, 16 layers, latent and differential
+    attention in turn, feed-forward 8192, vocabulary 128256, beside the Llama-3 decoder of the same width, depth,
+    feed-forward size and vocabulary.  Value: decode tokens/s at batch 64 behind 1024-token prompts."""
+    nb, dl = pkg.nibelorn, pkg.decode_loop
+    latent, differential, cfg = nibelorn_layers(nb)
+    llama = dl.DecoderConfig()
+    line = bench_decoders({
+        "nibelorn": (nb.NibelornDecoder, cfg, lambda: nb.init_weights(cfg, 42 + rank, dev)),
+        "llama3": (dl.Llama3Decoder, llama, lambda: {k: v.to(dev) for k, v in dl.init_weights(llama, 42 + rank).items()})},
+        ext, dev, rank, world)
     return {
-        "metric": "Nibelorn decode tokens/sec", "value": head["decode_tokens_per_s"], "unit": "tokens/s", "n_gpus": world,
-        "steps": long - 2, "warmup": short, "ms_per_step": head["decode_ms_per_step"], "higher_is_better": True, "scaling": "weak",
-        "vs_baseline": None, "dtype": "bf16", "data": "synthetic",
+        "metric": "Nibelorn decode tokens/sec", **line,
         "config": {"model": "Nibelorn, random weights: width 2048, 16 layers (latent attention 16 x (128 + 64), rank 512, values 128; "
                             "differential attention 16 / 4 heads, 2 x 64, values 128), feed-forward 8192, vocabulary 128256",
                    "beside": "Llama-3 decoder of equal width, depth, feed-forward size and vocabulary (32 / 8 heads of 64)",
                    "global_batch": 64 * world, "seq_len": 1024, "parallelism": "replicas x%d" % world,
                    "l2": "weights and cache of a step exceed L2"},
-        "models": models, "kernels": mixer_kernel_table(ext, pkg, dev, latent, differential) if rank == 0 else None,
-        "e2e": e2e,
+        "kernels": mixer_kernel_table(ext, pkg, dev, latent, differential) if rank == 0 else None,
         # embedding, 16 x (cache write, attention, two norms, gelu), token choice; the split merges come on top
-        "gpu_launches": (long - 2) * (1 + 16 * 5 + 1), "clocks": sampler.summary(),
+        "gpu_launches": line["steps"] * (1 + 16 * 5 + 1),
     }
 
 
-def mixer_kernel_table(ext, pkg, dev, latent, differential):
-    """Roofline of every mixer kernel beside the Llama-3 kernel that does the like: fraction of the measured peak each."""
-    mx = pkg.mixers
-    hbm, _ = hbm_peak()
-    peaks = REPO / "MEASURED_PEAKS.json"
-    tensor = float(json.loads(peaks.read_text())["bf16_tflops"]) if peaks.exists() else 1590.0
-    bf16 = dict(dtype=torch.bfloat16, device=dev)
-    table = []
+def rupotar_config(ru):
+    """Twelve layers, four of them run twice: 16 layer runs, of which eight attend, four run each recurrence; the experts of
+    a token together are as large as the dense feed-forward of 8192."""
+    windowed = ru.Attention(heads=16, kv_heads=4, dim=128, vdim=128, scale=128 ** -0.5, window=1024, keep_first=64)
+    full = ru.Attention(heads=16, kv_heads=4, dim=128, vdim=128, scale=128 ** -0.5)
+    delta, mix = ru.ChannelDelta(heads=16, kv_heads=16, dim=128, vdim=128, taps=4), ru.TimeMix(heads=32, dim=64)
+    dense, experts = ru.Dense(8192), ru.Experts(ff=2048, limit=7.0, experts=16, top=4)
+    mixers = [windowed, delta, full, mix, windowed, delta, windowed, mix, full, delta, windowed, mix]
+    layers = tuple(ru.Layer(m, experts if i % 2 else dense) for i, m in enumerate(mixers))
+    return ru.RupotarConfig(128256, 2048, 1e-5, 45.0, layers, ru.Loop(4, 8, 2))
 
-    def us(step, n):
-        run = graph_runner(step, n, dev)
+
+def bench_rupotar(args, ext, pkg, dev, rank, world):
+    """The Rupotar decoder (random weights) at a 1B model's layer sizes (`rupotar_config`) beside the Nibelorn decoder of equal
+    width, number of layer runs, active feed-forward size and vocabulary.  Value: decode tokens/s at batch 64 behind
+    1024-token prompts."""
+    ru, nb = pkg.rupotar, pkg.nibelorn
+    cfg, near = rupotar_config(ru), nibelorn_layers(nb)[2]
+    line = bench_decoders({
+        "rupotar": (ru.RupotarDecoder, cfg, lambda: ru.init_weights(cfg, 42 + rank, dev, rank=128)),
+        "nibelorn": (nb.NibelornDecoder, near, lambda: nb.init_weights(near, 42 + rank, dev))}, ext, dev, rank, world)
+    return {
+        "metric": "Rupotar decode tokens/sec", **line,
+        "config": {"model": "Rupotar, random weights: width 2048, 12 layers, four of them twice (attention 16 / 4 heads of 128, window 1024 and 64 "
+                            "kept or none; delta rule 16 heads 128 x 128, 4 taps; time mixing 32 heads of 64), dense 8192 or 4 of 16 "
+                            "experts of 2048, vocabulary 128256",
+                   "beside": "Nibelorn decoder of equal width, layer runs, active feed-forward size and vocabulary",
+                   "global_batch": 64 * world, "seq_len": 1024, "parallelism": "replicas x%d" % world,
+                   "l2": "weights and cache of a step exceed L2"},
+        "kernels": rupotar_kernel_table(ext, pkg, dev, cfg) if rank == 0 else None,
+        # per step: embedding, token choice; per run two norms; per attention two, delta three, time mixing three (token shift, tanh,
+        # scan); per dense one, experts four; per pass of the loop one more norm
+        "gpu_launches": line["steps"] * (2 + 16 * 2 + 8 * 2 + 4 * 3 + 4 * 3 + 8 * 1 + 8 * 4 + 2),
+    }
+
+
+class KernelTable:
+    """Rows of (kernel, shape, time, fraction of its measured roofline) beside the like kernel of another model."""
+
+    def __init__(self, dev):
+        self.dev, self.rows = dev, []
+        peaks = REPO / "MEASURED_PEAKS.json"
+        self.byte = hbm_peak()[0] * 1e3                                     # bytes, flops per microsecond
+        self.flop = (float(json.loads(peaks.read_text())["bf16_tflops"]) if peaks.exists() else 1590.0) * 1e6
+
+    def us(self, step, n):
+        run = graph_runner(step, n, self.dev)
         run.prepare(n)
         run(4 * n)
         times = []
@@ -1150,17 +1203,160 @@ def mixer_kernel_table(ext, pkg, dev, latent, differential):
             times.append(start.elapsed_time(end) * 1e3 / (8 * n))
         return sorted(times)[2]
 
+    @staticmethod
     def sets(bytes_each):
         return int(max(2, min(24, 4e8 // bytes_each + 1)))   # rotating inputs beyond L2
 
-    def row(name, shape, ours, like_name, like):
+    def row(self, name, shape, ours, like_name, like):
         """ours, like: (microseconds, bytes or flops, peak per microsecond)"""
         frac = [work / t / peak for t, work, peak in (ours, like)]
-        table.append({"kernel": name, "shape": shape, "us": ours[0], "frac": frac[0], "like": like_name, "like_us": like[0],
-                      "like_frac": frac[1], "frac_over_like": frac[0] / frac[1]})
+        self.rows.append({"kernel": name, "shape": shape, "us": ours[0], "frac": frac[0], "like": like_name, "like_us": like[0],
+                          "like_frac": frac[1], "frac_over_like": frac[0] / frac[1]})
         torch.cuda.empty_cache()
 
-    byte, flop = hbm * 1e3, tensor * 1e6   # bytes, flops per microsecond
+
+def rupotar_kernel_table(ext, pkg, dev, cfg):
+    """Every kernel of the Rupotar decoder beside the kernel of the Nibelorn decoder that does the like.  Bytes: inputs and
+    outputs once; the scans over prompts against the fp32 rate of the device (`fma`), which is what they run on."""
+    ru, mx, tab = pkg.rupotar, pkg.mixers, KernelTable(dev)
+    us, sets, row, byte, flop = tab.us, tab.sets, tab.row, tab.byte, tab.flop
+    fma = torch.cuda.get_device_properties(dev).multi_processor_count * 128 * 2 * 1.965e3      # fp32 flops per microsecond at the top clock
+    bf16, f32 = dict(dtype=torch.bfloat16, device=dev), dict(dtype=torch.float32, device=dev)
+    _, differential, _ = nibelorn_layers(pkg.nibelorn)
+    att, delta, mix, ex = cfg.layers[2].mixer, cfg.layers[1].mixer, cfg.layers[3].mixer, cfg.layers[1].ff
+    E, eps = cfg.width, 1e-5
+
+    def attention(m, B, T, S, n, window=0, keep=0):
+        q, o = torch.randn(B, T, m.heads, m.dim, **bf16), torch.empty(B, T, m.heads, m.vdim, **bf16)
+        k, v = [torch.randn(B, S, m.kv_heads, m.dim, **bf16) for _ in range(n)], [torch.randn(B, S, m.kv_heads, m.vdim, **bf16) for _ in range(n)]
+        pos = torch.full((B,), S - T, dtype=torch.int32, device=dev)
+        return us(lambda i: mx.attention(q, k[i], v[i], o, pos, scale=m.scale, start_pos=S - T if T > 1 else -1, window=window, keep_first=keep,
+                                         bias_range=ru.SLOPE_RANGE, sink=True), n)
+
+    def like_attention(m, B, T, S, n):
+        q, o, gate = torch.randn(B, T, m.heads, 2 * m.dim, **bf16), torch.empty(B, T, m.heads, m.vdim, **bf16), torch.randn(B, T, m.heads, **bf16)
+        k, v = [torch.randn(B, S, m.kv_heads, 2 * m.dim, **bf16) for _ in range(n)], [torch.randn(B, S, m.kv_heads, m.vdim, **bf16) for _ in range(n)]
+        pos = torch.full((B,), S - T, dtype=torch.int32, device=dev)
+        return us(lambda i: mx.attention(q, k[i], v[i], o, pos, maps=2, scale=m.scale, softcap=50.0, temp_coef=0.3, temp_every=256.0, gate=gate,
+                                         lambda_=0.5, post=0.5, eps=eps, start_pos=S - T if T > 1 else -1), n)
+
+    def scan(kind, B, T, n):
+        H, D, V = (delta.heads, delta.dim, delta.vdim) if kind == 0 else (mix.heads, mix.dim, mix.dim)
+        t = torch.float32 if kind == 0 else torch.bfloat16
+        qk = [torch.randn(B, T, 2, H, D, dtype=t, device=dev) * D ** -0.5 for _ in range(n)]
+        v, gate = [torch.randn(B, T, H, V, **bf16) for _ in range(n)], torch.randn(B, T, H, V, **bf16)
+        g = [(torch.rand(B, T, H, D, device=dev) * 0.1 + 0.9 if kind == 0 else torch.randn(B, T, H, D, device=dev) - 3).to(t) for _ in range(n)]
+        state = [torch.zeros(B, H, D, V, device=dev) for _ in range(n)]
+        pos = torch.full((B,), 7, dtype=torch.int32, device=dev)
+        kw = dict(beta=torch.rand(B, T, H, device=dev)) if kind == 0 else dict(bonus=torch.rand(H, D, device=dev), g_bias=torch.zeros(H * D, device=dev))
+        norm = torch.ones(H, V, device=dev)
+        return us(lambda i: mx.recurrent_scan(qk[i][:, :, 0], qk[i][:, :, 1], v[i], g[i], state[i], pos, norm, gate, act=kind, eps=eps, **kw), n)
+
+    for B, S in ((64, 1024), (64, 2048), (8, 8192), (1, 65536)):
+        n = sets(B * S * att.kv_heads * 2 * att.dim * 2)
+        t = attention(att, B, 1, S, n)
+        like = like_attention(differential, B, 1, S, n), B * S * 4 * 256 * 2, byte
+        row("decode attention", f"B={B} keys={S}", (t, B * S * att.kv_heads * 2 * att.dim * 2, byte), "differential decode attention", like)
+        if S > 1024:
+            t = attention(att, B, 1, S, n, 1024, 64)
+            row("decode attention, window 1024 + 64", f"B={B} keys={S}", (t, B * 1088 * att.kv_heads * 2 * att.dim * 2, byte),
+                f"differential decode attention, keys={S}", like)
+    for B, T in ((4, 2048), (1, 8192)):
+        pairs = B * T * (T + 1) / 2
+        like = like_attention(differential, B, T, T, 4), 4 * 16 * pairs * (64 + 128), flop
+        row("prefill attention", f"B={B} T={T}", (attention(att, B, T, T, 4), 4 * 16 * pairs * 128, flop), "differential prefill attention", like)
+        seen = B * sum(min(t + 1, 1024) + min(64, max(0, t + 1 - 1024)) for t in range(T))
+        row("prefill attention, window 1024 + 64", f"B={B} T={T}", (attention(att, B, T, T, 4, 1024, 64), 4 * 16 * seen * 128, flop),
+            "differential prefill attention", like)
+        ours = scan(0, B, T, 2), B * T * delta.heads * delta.dim * delta.vdim * 7, fma
+        row("delta rule scan (+ norm, gate)", f"B={B} T={T}", ours, "differential prefill attention", like)
+        ours = scan(1, B, T, 2), B * T * mix.heads * mix.dim * mix.dim * 5, fma
+        row("time mixing scan (+ norm, gate)", f"B={B} T={T}", ours, "differential prefill attention", like)
+    for B, S in ((64, 1024), (8, 8192), (1, 65536)):
+        like = like_attention(differential, B, 1, S, sets(B * S * 4 * 256 * 2)), B * S * 4 * 256 * 2, byte
+        bytes_ = B * delta.heads * delta.dim * delta.vdim * 8
+        row("delta rule step (+ norm, gate)", f"B={B}", (scan(0, B, 1, sets(bytes_)), bytes_, byte), f"differential decode attention, keys={S}", like)
+        bytes_ = B * mix.heads * mix.dim * mix.dim * 8
+        row("time mixing step (+ norm, gate)", f"B={B}", (scan(1, B, 1, sets(bytes_)), bytes_, byte), f"differential decode attention, keys={S}", like)
+    for B, T in ((64, 1), (4, 2048)):
+        N = B * T
+        pos = torch.zeros(B, dtype=torch.int32, device=dev)
+        n = sets(N * E * 12)
+        w = [torch.ones(E, device=dev) for _ in range(4)]
+        x, y = [torch.randn(N, E, device=dev) for _ in range(n)], [torch.randn(N, E, **bf16) for _ in range(n)]
+        like = us(lambda i: mx.add_dyn_tanh(y[i], x[i], w[0], w[1], 0.5), n), N * E * 12, byte
+        row("residual_norm (two layer norms)", f"{N} x {E}",
+            (us(lambda i: mx.residual_norm(y[i], x[i], dtype=torch.bfloat16, post=(w[0], w[1]), pre=(w[2], w[3]), eps=eps), n), N * E * 12, byte),
+            "add_dyn_tanh", like)
+        del y
+        n = sets(N * E * (8 + 2 * ex.top))
+        y = [torch.randn(N * ex.top, E, **bf16) for _ in range(n)]
+        parts, pw = torch.randperm(N * ex.top, device=dev).int().view(N, ex.top), torch.rand(N, ex.top, device=dev)
+        row("residual_norm (two layer norms, four experts)", f"{N} x {E}",
+            (us(lambda i: mx.residual_norm(y[i], x[i], dtype=torch.bfloat16, post=(w[0], w[1]), pre=(w[2], w[3]), eps=eps, part_rows=parts,
+                                           part_weights=pw), n), N * E * (10 + 2 * ex.top), byte), "add_dyn_tanh", like)
+        del x, y
+        n = sets(N * 8192 * 4)
+        gu, z = [torch.randn(N, 2 * 8192, **bf16) for _ in range(n)], [torch.randn(N, 8192, **bf16) for _ in range(n)]
+        like = us(lambda i: mx.gelu_(z[i]), n), N * 8192 * 4, byte
+        row("gated_act", f"{N} x {8192}", (us(lambda i: mx.gated_act(gu[i]), n), N * 8192 * 6, byte), "gelu", like)
+        del gu, z
+        n = sets(N * 3072 * 2)
+        m, d = att, differential
+        qkv = [torch.randn(B, T, (m.heads + 2 * m.kv_heads) * m.dim, **bf16) for _ in range(n)]
+        ck, cv = torch.zeros(B, T + 8, m.kv_heads, m.dim, **bf16), torch.zeros(B, T + 8, m.kv_heads, m.vdim, **bf16)
+        qw, kw = torch.ones(m.heads * m.dim, device=dev), torch.ones(m.kv_heads * m.dim, device=dev)
+        t = us(lambda i: mx.qk_norm_cache(qkv[i], m.heads * m.dim, m.kv_heads * m.dim, qw, kw, eps, ck, cv, pos), n)
+        lat = nibelorn_layers(pkg.nibelorn)[0]
+        C, R, H, D = lat.kv_rank, lat.rot_dim, lat.heads, lat.dim
+        qd = [torch.randn(B, T, H * (D + R) + C + R, **bf16) for _ in range(n)]
+        cache, rot, nw = torch.zeros(B, T + 8, C + R, **bf16), pkg.rope_table.rotation_table(R, T + 8, 1e4).to(dev), torch.ones(C, device=dev)
+        like_rows = us(lambda i: mx.latent_cache(qd[i], rot, nw, eps, cache, pos, H, D, R, C), n), N * (H * R + C + R) * 4, byte
+        row("qk_norm_cache", f"{N} tokens", (t, N * 3072 * 4, byte), "latent_cache", like_rows)
+        del qkv, qd
+        h, last, mu = [torch.randn(B, T, E, **bf16) for _ in range(n)], torch.zeros(B, E, **bf16), torch.rand(5, E, device=dev)
+        row("token_shift", f"{N} x {E}", (us(lambda i: mx.token_shift(h[i], mu, last, pos), n), N * E * 12, byte), "gelu", like)
+        H, D, V = delta.heads, delta.dim, delta.vdim
+        n = sets(N * H * D * 26)
+        p = [torch.randn(B, T, delta.channels + H, **bf16) for _ in range(n)]
+        a, conv, tail = [torch.randn(B, T, H * D, **bf16) for _ in range(n)], torch.randn(4, delta.channels, device=dev), torch.zeros(B, 3, delta.channels, **bf16)
+        al, dt = torch.zeros(H, device=dev), torch.zeros(H * D, device=dev)
+        t = us(lambda i: mx.delta_inputs(p[i], p[i][..., -H:], a[i], conv, al, dt, tail, pos, H, H, D, V), n)
+        tail_bytes = B * 3 * delta.channels * 2
+        row("delta_inputs", f"{N} tokens", (t, N * H * D * (8 + 12 + 2) + tail_bytes, byte), "latent_cache", like_rows)
+        del p, a
+        n = sets(N * E * 2)
+        h = [torch.randn(N, E, **bf16) for _ in range(n)]
+        router, rb = torch.randn(ex.experts, E, **bf16), torch.zeros(ex.experts, device=dev)
+        t = us(lambda i: mx.moe_route(h[i], router, rb, ex.top), n)
+        row("moe_route", f"{N} x {ex.experts}", (t, N * E * 2 + ex.experts * E * 2, byte), "gelu", like)
+        experts, ranks, _, counts = mx.moe_route(h[0], router, rb, ex.top)
+        row("moe_gather", f"{N} x {ex.top}", (us(lambda i: mx.moe_gather(h[i], experts, ranks, counts), n), N * E * 2 * (1 + ex.top), byte),
+            "latent_cache", like_rows)
+        xs, _ = mx.moe_gather(h[0], experts, ranks, counts)
+        gu, down = [torch.randn(ex.experts, 2, ex.ff, E, **bf16) for _ in range(4)], [torch.randn(ex.experts, E, ex.ff, **bf16) for _ in range(4)]
+        act = mx.moe_gemm(xs, gu[0], counts, limit=ex.limit)
+        wl, wd = [torch.randn(2 * 8192, E, **bf16) for _ in range(4)], [torch.randn(E, 8192, **bf16) for _ in range(4)]
+        hl = torch.randn(N, 8192, **bf16)
+
+        def work(K, cols, tokens, matrices):
+            return (2 * tokens * K * cols, flop) if N > 512 else (matrices * K * cols * 2 + tokens * (K + cols) * 2, byte)
+
+        t, like_t = us(lambda i: mx.moe_gemm(xs, gu[i], counts, limit=ex.limit), 4), us(lambda i: torch.mm(h[0], wl[i].t()), 4)
+        used = int((counts > 0).sum())
+        row("moe_gemm gate, up (+ activation)", f"{N} tokens", (t, *work(E, 2 * ex.ff, N * ex.top, used)), "cuBLAS, dense up of 16384", (like_t, *work(E, 16384, N, 1)))
+        t, like_t = us(lambda i: mx.moe_gemm(act, down[i], counts), 4), us(lambda i: torch.mm(hl, wd[i].t()), 4)
+        row("moe_gemm down", f"{N} tokens", (t, *work(ex.ff, E, N * ex.top, used)), "cuBLAS, dense down of 8192", (like_t, *work(8192, E, N, 1)))
+        del gu, down, wl, wd
+    return tab.rows
+
+
+def mixer_kernel_table(ext, pkg, dev, latent, differential):
+    """Roofline of every mixer kernel beside the Llama-3 kernel that does the like: fraction of the measured peak each."""
+    mx = pkg.mixers
+    tab = KernelTable(dev)
+    us, sets, row, byte, flop = tab.us, tab.sets, tab.row, tab.byte, tab.flop
+    bf16 = dict(dtype=torch.bfloat16, device=dev)
     C, R, H, D, V = latent.kv_rank, latent.rot_dim, latent.heads, latent.dim, latent.vdim
     G, d, Hd, Vd = differential.kv_heads, differential.dim, differential.heads, differential.vdim
 
@@ -1240,7 +1436,7 @@ def mixer_kernel_table(ext, pkg, dev, latent, differential):
         ck, cv = torch.zeros(B, T + 8, G, 2 * d, **bf16), torch.zeros(B, T + 8, G, Vd, **bf16)
         t = us(lambda i: mx.kv_cache_write(pk[i], 2 * Hd * d, 2 * (Hd + G) * d, ck, cv, pos), n)
         row("kv_cache_write", f"{N} tokens", (t, N * G * (2 * d + Vd) * 4, byte), "rot_embed_kv_cache", like)
-    return table
+    return tab.rows
 
 
 def time_sampling_step(ext, dev, B, vocab):
