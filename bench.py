@@ -1327,10 +1327,10 @@ def rupotar_kernel_table(ext, pkg, dev, cfg):
         del p, a
         n = sets(N * E * 2)
         h = [torch.randn(N, E, **bf16) for _ in range(n)]
-        router, rb = torch.randn(ex.experts, E, **bf16), torch.zeros(ex.experts, device=dev)
-        t = us(lambda i: mx.moe_route(h[i], router, rb, ex.top), n)
-        row("moe_route", f"{N} x {ex.experts}", (t, N * E * 2 + ex.experts * E * 2, byte), "gelu", like)
-        experts, ranks, _, counts = mx.moe_route(h[0], router, rb, ex.top)
+        logits, rb = torch.randn(N, ex.experts, device=dev), torch.zeros(ex.experts, device=dev)
+        t = us(lambda i: mx.moe_route(logits, rb, ex.top), 8)
+        row("moe_route", f"{N} x {ex.experts}", (t, N * ex.experts * 4 + N * ex.top * 12, byte), "latent_cache", like_rows)
+        experts, ranks, _, counts = mx.moe_route(logits, rb, ex.top)
         row("moe_gather", f"{N} x {ex.top}", (us(lambda i: mx.moe_gather(h[i], experts, ranks, counts), n), N * E * 2 * (1 + ex.top), byte),
             "latent_cache", like_rows)
         xs, _ = mx.moe_gather(h[0], experts, ranks, counts)

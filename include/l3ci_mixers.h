@@ -132,12 +132,11 @@ typedef struct l3ci_recurrent_scan_args {
 
 L3CI_API int l3ci_recurrent_scan(const l3ci_recurrent_scan_args* args);
 
-/* Mixture of experts.  Route: logits = router h + bias in fp32 (router: dtype [E, width], bias fp32), the `top` largest of a
- * token (ties: the smaller index), weights = softmax over these; experts, ranks int32 [rows, top] (rank: place of the pair
- * among the pairs of its expert), weights fp32.  counts int32 [E] is set to the experts' pairs. */
-L3CI_API int l3ci_moe_route(const void* h, const void* router, const float* bias, int32_t* experts, int32_t* ranks,
-                            float* weights, int32_t* counts, int64_t rows, int64_t width, int32_t n_experts, int32_t top,
-                            int32_t dtype, l3ci_stream_t stream);
+/* Mixture of experts.  Route: of the fp32 logits [rows, E] + bias [E] the `top` largest of a token (ties: the smaller index),
+ * weights = softmax over these; experts, ranks int32 [rows, top] (rank: place of the pair among the pairs of its expert),
+ * weights fp32.  counts int32 [E] is set to the experts' pairs. */
+L3CI_API int l3ci_moe_route(const float* logits, const float* bias, int32_t* experts, int32_t* ranks, float* weights,
+                            int32_t* counts, int64_t rows, int32_t n_experts, int32_t top, l3ci_stream_t stream);
 /* Rows sorted by expert: out[at] = h[row], at = (sum of counts of smaller experts) + rank; part_rows[row, j] = at. */
 L3CI_API int l3ci_moe_gather(const void* h, const int32_t* experts, const int32_t* ranks, const int32_t* counts, void* out,
                              int32_t* part_rows, int64_t rows, int64_t width, int32_t n_experts, int32_t top, int32_t dtype,

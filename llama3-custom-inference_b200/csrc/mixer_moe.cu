@@ -1,9 +1,8 @@
 // Mixture of experts: routing, sorting of the token rows by expert, and the plain form of the experts' products
 // (mixer_moe_tc.cu has the tensor-core form).
 //
-// route: a CTA takes TOKENS tokens, its warps the experts in turn; logits in fp32, then a warp picks a token's experts.  The
-// place of a (token, expert) pair among its expert's pairs is counted in shared memory per CTA and placed with one atomic per
-// CTA and expert.  The order of an expert's rows is whatever that gives: a row's result does not depend on its place.
+// route: a warp picks a token's experts from its fp32 logits.  The place of a (token, expert) pair among its expert's pairs is
+// counted in shared memory per CTA and placed with one atomic per CTA and expert.  The order of an expert's rows is whatever that gives: a row's result does not depend on its place.
 #include <cuda_bf16.h>
 #include <cuda_runtime.h>
 
@@ -16,80 +15,59 @@ namespace l3ci {
 namespace {
 
 constexpr int kRouteWarps = 8;
-constexpr int kPer = 2;            // experts of a warp at a time
 
-template <typename S, int VEC, int TOKENS>
+// Order of the floats as unsigned numbers; NaN is below every number.
+__device__ __forceinline__ unsigned ordered(float z) {
+  const unsigned u = __float_as_uint(z);
+  return z != z ? 0u : u & 0x80000000u ? ~u : u | 0x80000000u;
+}
+
 __global__ void __launch_bounds__(32 * kRouteWarps)
-moe_route_kernel(const S* __restrict__ h, const S* __restrict__ router, const float* __restrict__ bias, int* __restrict__ experts,
-                 int* __restrict__ ranks, float* __restrict__ weights, int* __restrict__ counts, long long rows, int width, int E, int top) {
+moe_route_kernel(const float* __restrict__ logits, const float* __restrict__ bias, int* __restrict__ experts, int* __restrict__ ranks,
+                 float* __restrict__ weights, int* __restrict__ counts, long long rows, int tokens, int E, int top) {
   extern __shared__ float sh[];
-  float* logit = sh;                                              // [TOKENS][E]
-  int* count = reinterpret_cast<int*>(logit + TOKENS * E);        // [E], then the expert's first rank of this CTA
-  int* chosen = count + E;                                        // [TOKENS][top]
-  int* place = chosen + TOKENS * top;                             // [TOKENS][top]
+  float* row = sh;                                                // [warps][E]
+  int* count = reinterpret_cast<int*>(row + kRouteWarps * E);     // [E], then the expert's first rank of this CTA
+  int* chosen = count + E;                                        // [tokens][top]
+  int* place = chosen + tokens * top;                             // [tokens][top]
+  float* weight = reinterpret_cast<float*>(place + tokens * top);
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   for (int e = tid; e < E; e += blockDim.x) count[e] = 0;
+  __syncthreads();
   pdl_wait();
   pdl_launch_dependents();
-  const long long row0 = (long long)blockIdx.x * TOKENS;
-  const int n = (int)min((long long)TOKENS, rows - row0);
-  for (int e0 = warp * kPer; e0 < E; e0 += kRouteWarps * kPer) {
-    float acc[kPer][TOKENS];
-#pragma unroll
-    for (int i = 0; i < kPer; ++i)
-#pragma unroll
-      for (int t = 0; t < TOKENS; ++t) acc[i][t] = 0.f;
-    for (int c = lane * VEC; c < width; c += 32 * VEC) {
-      float w[kPer][VEC];
-#pragma unroll
-      for (int i = 0; i < kPer; ++i) load_vec<S, VEC>(router + (long long)min(e0 + i, E - 1) * width + c, w[i]);
-#pragma unroll
-      for (int t = 0; t < TOKENS; ++t) {
-        float x[VEC];
-        load_vec<S, VEC>(h + (row0 + min(t, n - 1)) * width + c, x);
-#pragma unroll
-        for (int i = 0; i < kPer; ++i)
-#pragma unroll
-          for (int k = 0; k < VEC; ++k) acc[i][t] = fmaf(w[i][k], x[k], acc[i][t]);
-      }
-    }
-#pragma unroll
-    for (int i = 0; i < kPer; ++i)
-#pragma unroll
-      for (int t = 0; t < TOKENS; ++t) {
-        const float z = group_sum<kWarp>(acc[i][t]);
-        if (lane == 0 && e0 + i < E) logit[t * E + e0 + i] = z + bias[e0 + i];
-      }
-  }
-  __syncthreads();
+  const long long row0 = (long long)blockIdx.x * tokens;
+  const int n = (int)min((long long)tokens, rows - row0);
+  float* z = row + warp * E;
   for (int t = warp; t < n; t += kRouteWarps) {
-    float* z = logit + t * E;
+    for (int e = lane; e < E; e += 32) z[e] = logits[(row0 + t) * E + e] + bias[e];
+    __syncwarp();
     float first = 0.f, sum = 0.f;
     for (int j = 0; j < top; ++j) {
-      float best = -INFINITY;
-      int at = 0x7fffffff;
-      for (int e = lane; e < E; e += 32)
-        if (z[e] > best) { best = z[e]; at = e; }                // NaN is never chosen before a number
-#pragma unroll
-      for (int m = 16; m >= 1; m >>= 1) {
-        const float ob = __shfl_xor_sync(kFullMask, best, m);
-        const int oa = __shfl_xor_sync(kFullMask, at, m);
-        if (ob > best || (ob == best && oa < at)) { best = ob; at = oa; }
+      // the lane's largest logit that is not taken (taken ones are NaN), then the warp's; ties: the smaller index
+      unsigned best = 0u;
+      int at = E;
+      for (int e = lane; e < E; e += 32) {
+        const unsigned o = ordered(z[e]);
+        if (o > best) { best = o; at = e; }
       }
-      if (at >= E) at = j;                                        // nothing comparable left: any place within bounds
-      if (j == 0) first = best;
-      const float p = expf(best - first);
+      const unsigned most = __reduce_max_sync(kFullMask, best);
+      at = __reduce_min_sync(kFullMask, best == most ? at : E);
+      if (at >= E) at = j;                                        // nothing but NaN left: any place within bounds
+      const float v = z[at];
+      if (j == 0) first = v;
+      const float p = expf(v - first);
       sum += p;
+      __syncwarp();
       if (lane == 0) {
-        z[at] = -INFINITY;
+        z[at] = __int_as_float(0x7fffffff);
         chosen[t * top + j] = at;
         place[t * top + j] = atomicAdd(count + at, 1);
-        weights[(row0 + t) * top + j] = p;
+        weight[t * top + j] = p;
       }
       __syncwarp();
     }
-    if (lane == 0)
-      for (int j = 0; j < top; ++j) weights[(row0 + t) * top + j] /= sum;
+    for (int j = lane; j < top; j += 32) weights[(row0 + t) * top + j] = weight[t * top + j] / sum;
   }
   __syncthreads();
   for (int e = tid; e < E; e += blockDim.x)
@@ -207,34 +185,25 @@ int choose(const l3ci_moe_gemm_args* a) {
 
 extern "C" {
 
-int l3ci_moe_route(const void* h, const void* router, const float* bias, int32_t* experts, int32_t* ranks, float* weights, int32_t* counts,
-                   int64_t rows, int64_t width, int32_t E, int32_t top, int32_t dtype, l3ci_stream_t stream_) {
+int l3ci_moe_route(const float* logits, const float* bias, int32_t* experts, int32_t* ranks, float* weights, int32_t* counts, int64_t rows,
+                   int32_t E, int32_t top, l3ci_stream_t stream_) {
   using namespace l3ci;
   clear_error();
-  if (rows < 0 || rows > 0x7fffffffLL / 8 || width <= 0 || width > 0x3fffffffLL || E <= 0 || E > kMaxExperts || top <= 0 || top > E ||
-      rows * top > 0x7fffffffLL || (dtype != L3CI_BF16 && dtype != L3CI_F32))
-    return fail(L3CI_ERR_INVALID, "moe_route: rows=%lld width=%lld experts=%d top=%d", (long long)rows, (long long)width, E, top);
+  if (rows < 0 || rows > 0x7fffffffLL / 8 || E <= 0 || E > kMaxExperts || top <= 0 || top > E || rows * top > 0x7fffffffLL)
+    return fail(L3CI_ERR_INVALID, "moe_route: rows=%lld experts=%d top=%d", (long long)rows, E, top);
   if (!counts) return fail(L3CI_ERR_INVALID, "moe_route: null pointer");
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream_);
   L3CI_CUDA_TRY(cudaMemsetAsync(counts, 0, sizeof(int32_t) * E, s));
   if (rows == 0) return L3CI_OK;
-  if (!h || !router || !bias || !experts || !ranks || !weights) return fail(L3CI_ERR_INVALID, "moe_route: null pointer");
+  if (!logits || !bias || !experts || !ranks || !weights) return fail(L3CI_ERR_INVALID, "moe_route: null pointer");
   const int sms = sm_count() > 0 ? sm_count() : 148;
-  const bool many = rows >= 4LL * sms && E <= 256 && top <= 64;   // (the tokens' logits fit 48 KB of shared memory)
-  auto typed = [&](auto zero) -> int {
-    using S = decltype(zero);
-    constexpr int kVec = 16 / sizeof(S);
-    const bool v = width % kVec == 0 && aligned16(h) && aligned16(router);
-    auto go = [&](auto kernel, int tokens) -> int {
-      const size_t smem = sizeof(float) * ((size_t)tokens * E + E + 2 * (size_t)tokens * top);
-      L3CI_LAUNCH("moe_route_kernel", kernel, dim3((unsigned)((rows + tokens - 1) / tokens)), dim3(32 * kRouteWarps), smem, s,
-                  static_cast<const S*>(h), static_cast<const S*>(router), bias, experts, ranks, weights, counts, (long long)rows, (int)width, E, top);
-      return L3CI_OK;
-    };
-    if (many) return v ? go(moe_route_kernel<S, kVec, 8>, 8) : go(moe_route_kernel<S, 1, 8>, 8);
-    return v ? go(moe_route_kernel<S, kVec, 1>, 1) : go(moe_route_kernel<S, 1, 1>, 1);
-  };
-  return dtype == L3CI_BF16 ? typed(__nv_bfloat16{}) : typed(float{});
+  int tokens = rows >= 16LL * sms ? 4 * kRouteWarps : rows >= kRouteWarps ? kRouteWarps : 1;
+  auto bytes = [&](int n) { return sizeof(float) * ((size_t)kRouteWarps * E + E + 3 * (size_t)n * top); };
+  while (tokens > 1 && bytes(tokens) > (48 << 10)) tokens /= 2;
+  if (bytes(tokens) > (48 << 10)) return fail(L3CI_ERR_UNSUPPORTED, "moe_route: experts=%d top=%d", E, top);
+  L3CI_LAUNCH("moe_route_kernel", moe_route_kernel, dim3((unsigned)((rows + tokens - 1) / tokens)), dim3(32 * kRouteWarps), bytes(tokens), s, logits,
+              bias, experts, ranks, weights, counts, (long long)rows, tokens, E, top);
+  return L3CI_OK;
 }
 
 int l3ci_moe_gather(const void* h, const int32_t* experts, const int32_t* ranks, const int32_t* counts, void* out, int32_t* part_rows,

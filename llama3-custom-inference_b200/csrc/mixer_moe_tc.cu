@@ -169,7 +169,7 @@ moe_tc_kernel(const __grid_constant__ CUtensorMap xmap, const __grid_constant__ 
 #pragma unroll
             for (int i = 0; i < 8; ++i) {
               f[i] = __uint_as_float(y[v * 8 + i]);
-              if (GATED) f[i] = gated_activation(f[i], __uint_as_float(z[v * 8 + i]), a.limit, a.alpha);
+              if (GATED) f[i] = gated_activation_fast(f[i], __uint_as_float(z[v * 8 + i]), a.limit, a.alpha);
             }
             *reinterpret_cast<uint4*>(dst + c + v * 8) = pack8(f);
           }

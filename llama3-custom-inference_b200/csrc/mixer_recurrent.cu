@@ -9,11 +9,14 @@
 // so that a token costs one reduction over the 8 lanes; k . q (and the bonus product of time mixing) is the same for all
 // columns and comes with the token.  Rows go two at a time through packed fp32 instructions.
 // Four producer warps stage the next tokens (convert, form decays, take the scalar products) in a ring of two chunks while
-// the others compute.  One token, all columns in the CTA: the head's output norm and gate are applied in place of the plain
-// store; otherwise head_norm_gate_kernel does it in a pass over the output rows.
+// the others compute; a chunk's loads are all in flight before the chunk ahead of it is handed over.  The head's output norm
+// and gate follow in a pass over the output rows (head_norm_gate_kernel).
 //
-// delta_inputs_kernel: convolution, activation, unit norms, step sizes and decays of all tokens at once; a warp per (token,
-// head) of one of q, k, v or the decay.
+// recurrent_step_kernel: one token.  A CTA per head streams the state through registers, four columns and every n-th row a
+// thread (whole rows per warp access), meets in shared memory for the two products, and applies norm and gate itself.
+//
+// delta_inputs_kernel: convolution, activation, unit norms, step sizes and decays of all tokens at once; a warp per run of
+// tokens and head of one of q, k, v or the decay.
 #include <cuda_bf16.h>
 #include <cuda_runtime.h>
 #include <math.h>
@@ -46,21 +49,48 @@ struct ScanParams {
   int vec;                       // q, k, g (and their fp32 companions) allow accesses of four elements
 };
 
+// Four channels from d on, zeros behind the last one (loaded from a place that exists, so that no load hangs on a branch).
 template <typename S>
 __device__ __forceinline__ float4 fetch4(const S* p, int d, int D, int vec) {
-  float f[4] = {0.f, 0.f, 0.f, 0.f};
+  float f[4];
   if (vec) {
-    if (d < D) load_vec<S, 4>(p + d, f);
+    load_vec<S, 4>(p + (d < D ? d : 0), f);
+#pragma unroll
+    for (int e = 0; e < 4; ++e) f[e] = d < D ? f[e] : 0.f;
   } else {
 #pragma unroll
-    for (int e = 0; e < 4; ++e)
-      if (d + e < D) f[e] = to_f32(p[d + e]);
+    for (int e = 0; e < 4; ++e) f[e] = to_f32(p[d + e < D ? d + e : 0]);
+#pragma unroll
+    for (int e = 0; e < 4; ++e) f[e] = d + e < D ? f[e] : 0.f;
   }
   return make_float4(f[0], f[1], f[2], f[3]);
 }
 
+// The convolution's carried inputs: row r of the tail becomes the input of token T - (taps - 1) + r.  Channel c of a sequence,
+// by one thread.
+template <typename S>
+__device__ __forceinline__ void move_tail(const l3ci_recurrent_scan_args& a, S* tail, const S* in, long long channels, long long c, bool fresh) {
+  const int rows = a.taps - 1;
+  for (int r = 0; r < rows; ++r) {
+    const int t = a.T - rows + r;
+    tail[r * channels + c] = t >= 0 ? in[t * a.conv_st + c] : fresh ? from_f32<S>(0.f) : tail[(r + a.T) * channels + c];
+  }
+}
+
+// Those of head h's values and, by the first head that reads them, of its queries and keys; `i` of `n` threads.
+template <typename S>
+__device__ __forceinline__ void move_tails(const l3ci_recurrent_scan_args& a, int b, int h, int i, int n, bool fresh) {
+  const int GD = a.G * a.D, R = a.H / a.G;
+  const long long channels = 2LL * GD + (long long)a.H * a.V;
+  S* tail = static_cast<S*>(a.tail) + b * a.tail_sb;
+  const S* in = static_cast<const S*>(a.conv_in) + (long long)b * a.T * a.conv_st;
+  for (int c = i; c < a.V; c += n) move_tail<S>(a, tail, in, channels, 2LL * GD + (long long)h * a.V + c, fresh);
+  if (h % R == 0)
+    for (int c = i; c < 2 * a.D; c += n) move_tail<S>(a, tail, in, channels, c < a.D ? (h / R) * a.D + c : GD + (h / R) * a.D + c - a.D, fresh);
+}
+
 // S: storage type of v, gate, out; Q: type of q, k, g.
-template <typename S, typename Q, int KIND, int NR, int C, bool FUSE>
+template <typename S, typename Q, int KIND, int NR, int C>
 __global__ void __launch_bounds__(kScanThreads) recurrent_scan_kernel(const __grid_constant__ ScanParams p) {
   constexpr int DP = NR * 8;
   extern __shared__ __align__(16) float smem[];
@@ -68,8 +98,7 @@ __global__ void __launch_bounds__(kScanThreads) recurrent_scan_kernel(const __gr
   const int cols = p.cols;
   const int stage_floats = kChunk * (3 * DP + cols + 2);
   float* stages = smem;
-  float* red = smem + kRing * stage_floats;                               // [kMaxConsumers]
-  uint64_t* bars = reinterpret_cast<uint64_t*>(red + kMaxConsumers);
+  uint64_t* bars = reinterpret_cast<uint64_t*>(smem + kRing * stage_floats);
   const uint32_t full0 = smem_u32(bars), empty0 = full0 + kRing * 8;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int split = blockIdx.x % p.splits, h = (blockIdx.x / p.splits) % a.H, b = blockIdx.x / (p.splits * a.H);
@@ -97,81 +126,86 @@ __global__ void __launch_bounds__(kScanThreads) recurrent_scan_kernel(const __gr
     const Q* gp = static_cast<const Q*>(a.g) + h * a.g_sh;
     const S* vp = static_cast<const S*>(a.v) + h * a.v_sh + col0;
     const int n_cols = min(cols, V - col0);
+    constexpr int kWide = (DP + 127) / 128;      // accesses of four channels per lane and row
+    constexpr int kCols = 4;                     // value columns per lane (a CTA has at most 128)
+    float4 q[kPerProducer][kWide], k[kPerProducer][kWide], g[kPerProducer][kWide];
+    float v[kPerProducer][kCols], beta[kPerProducer];
+    // all loads of this warp's tokens of chunk i (tokens behind the last one: the last one's, never used)
+    auto fetch = [&](int i) {
+#pragma unroll
+      for (int x = 0; x < kPerProducer; ++x) {
+        const long long row = row0 + min(i * kChunk + pw * kPerProducer + x, T - 1);
+#pragma unroll
+        for (int j = 0; j < kWide; ++j) {
+          const int d = j * 128 + lane * 4;
+          q[x][j] = fetch4<Q>(qp + row * a.qk_st, d, D, p.vec);
+          k[x][j] = fetch4<Q>(kp + row * a.qk_st, d, D, p.vec);
+          g[x][j] = fetch4<Q>(gp + row * a.g_st, d, D, p.vec);
+        }
+#pragma unroll
+        for (int c = 0; c < kCols; ++c) v[x][c] = to_f32(vp[row * a.v_st + min(c * 32 + lane, n_cols - 1)]);
+        beta[x] = KIND == kDelta ? a.beta[row * a.H + h] : 0.f;
+      }
+    };
+    float4 bonus[kWide], gb[kWide];
+    if (KIND == kTimeMix) {
+#pragma unroll
+      for (int j = 0; j < kWide; ++j) {
+        bonus[j] = fetch4<float>(a.bonus + h * D, j * 128 + lane * 4, D, p.vec);
+        gb[j] = fetch4<float>(a.g_bias + h * D, j * 128 + lane * 4, D, p.vec);
+      }
+    }
+    fetch(0);
     for (int i = 0; i < chunks; ++i) {
       const int s = i % kRing;
       if (i >= kRing && !mbar_wait_bounded(empty0 + s * 8, ((i / kRing) - 1) & 1)) { ok = false; break; }
       float* st = stages + s * stage_floats;
-      const int t0 = i * kChunk + pw * kPerProducer, n = min(kPerProducer, T - t0);
-      float scalar[kPerProducer];
-#pragma unroll
-      for (int x = 0; x < kPerProducer; ++x) scalar[x] = 0.f;
-#pragma unroll
-      for (int d0 = 0; d0 < DP; d0 += 128) {
-        const int d = d0 + lane * 4;
-        if (d >= DP) break;
-        float4 q[kPerProducer], k[kPerProducer], g[kPerProducer];
-#pragma unroll
-        for (int x = 0; x < kPerProducer; ++x) {
-          if (x >= n) continue;
-          const long long row = row0 + t0 + x;
-          q[x] = fetch4<Q>(qp + row * a.qk_st, d, D, p.vec);
-          k[x] = fetch4<Q>(kp + row * a.qk_st, d, D, p.vec);
-          g[x] = fetch4<Q>(gp + row * a.g_st, d, D, p.vec);
-        }
-        float4 bonus = make_float4(1.f, 1.f, 1.f, 1.f), gb = make_float4(0.f, 0.f, 0.f, 0.f);
-        if (KIND == kTimeMix) {
-          bonus = fetch4<float>(a.bonus + h * D, d, D, p.vec);
-          gb = fetch4<float>(a.g_bias + h * D, d, D, p.vec);
-        }
-#pragma unroll
-        for (int x = 0; x < kPerProducer; ++x) {
-          if (x >= n) continue;
-          if (KIND == kTimeMix) {
-            g[x].x = expf(-expf(g[x].x + gb.x));
-            g[x].y = expf(-expf(g[x].y + gb.y));
-            g[x].z = expf(-expf(g[x].z + gb.z));
-            g[x].w = expf(-expf(g[x].w + gb.w));
-          }
-          scalar[x] += q[x].x * k[x].x * bonus.x + q[x].y * k[x].y * bonus.y + q[x].z * k[x].z * bonus.z + q[x].w * k[x].w * bonus.w;
-          float* row = st + (pw * kPerProducer + x) * 3 * DP + d;
-          *reinterpret_cast<float4*>(row) = q[x];
-          *reinterpret_cast<float4*>(row + DP) = k[x];
-          *reinterpret_cast<float4*>(row + 2 * DP) = g[x];
-        }
-      }
       float* vs = st + kChunk * 3 * DP;
       float* sc = vs + kChunk * cols;
+      float scalar[kPerProducer];
 #pragma unroll
       for (int x = 0; x < kPerProducer; ++x) {
-        if (x >= n) continue;
         const int at = pw * kPerProducer + x;
-        const long long row = row0 + t0 + x;
-        for (int c = lane; c < cols; c += 32) vs[at * cols + c] = c < n_cols ? to_f32(vp[row * a.v_st + c]) : 0.f;
-        const float sum = group_sum<kWarp>(scalar[x]);
-        if (lane == 0) {
-          sc[at * 2] = sum;
-          sc[at * 2 + 1] = KIND == kDelta ? a.beta[row * a.H + h] : 0.f;
+        scalar[x] = 0.f;
+#pragma unroll
+        for (int j = 0; j < kWide; ++j) {
+          const int d = j * 128 + lane * 4;
+          const float4 qq = q[x][j], kk = k[x][j];
+          float4 gg = g[x][j];
+          if (KIND == kTimeMix) {
+            gg.x = expf(-expf(gg.x + gb[j].x));
+            gg.y = expf(-expf(gg.y + gb[j].y));
+            gg.z = expf(-expf(gg.z + gb[j].z));
+            gg.w = expf(-expf(gg.w + gb[j].w));
+            scalar[x] += qq.x * kk.x * bonus[j].x + qq.y * kk.y * bonus[j].y + qq.z * kk.z * bonus[j].z + qq.w * kk.w * bonus[j].w;
+          } else {
+            scalar[x] += qq.x * kk.x + qq.y * kk.y + qq.z * kk.z + qq.w * kk.w;
+          }
+          if (d < DP) {
+            float* row = st + at * 3 * DP + d;
+            *reinterpret_cast<float4*>(row) = qq;
+            *reinterpret_cast<float4*>(row + DP) = kk;
+            *reinterpret_cast<float4*>(row + 2 * DP) = gg;
+          }
+        }
+#pragma unroll
+        for (int c = 0; c < kCols; ++c)
+          if (c * 32 + lane < cols) vs[at * cols + c * 32 + lane] = c * 32 + lane < n_cols ? v[x][c] : 0.f;
+      }
+#pragma unroll
+      for (int x = 0; x < kPerProducer; ++x) scalar[x] = group_sum<kWarp>(scalar[x]);
+      if (lane == 0) {
+#pragma unroll
+        for (int x = 0; x < kPerProducer; ++x) {
+          sc[(pw * kPerProducer + x) * 2] = scalar[x];
+          sc[(pw * kPerProducer + x) * 2 + 1] = beta[x];
         }
       }
       __syncwarp();
       if (lane == 0) mbar_arrive(full0 + s * 8);
+      if (i + 1 < chunks) fetch(i + 1);
     }
-    // the convolution's last inputs: row r of the tail becomes the input of token T - (taps - 1) + r
-    if (a.tail && split == 0) {
-      const int rows = a.taps - 1, GD = a.G * D;
-      const long long C_all = 2LL * GD + (long long)a.H * V;
-      S* tail = static_cast<S*>(a.tail) + b * a.tail_sb;
-      const S* in = static_cast<const S*>(a.conv_in) + row0 * a.conv_st;
-      auto move = [&](long long c) {
-        for (int r = 0; r < rows; ++r) {
-          const int t = T - rows + r;
-          tail[r * C_all + c] = t >= 0 ? in[t * a.conv_st + c] : fresh ? from_f32<S>(0.f) : tail[(r + T) * C_all + c];
-        }
-      };
-      for (int c = pw * 32 + lane; c < V; c += 32 * kProducers) move(2LL * GD + (long long)h * V + c);
-      if (h % R == 0)
-        for (int c = pw * 32 + lane; c < 2 * D; c += 32 * kProducers) move(c < D ? (h / R) * D + c : GD + (h / R) * D + c - D);
-    }
+    if (a.tail && split == 0) move_tails<S>(a, b, h, pw * 32 + lane, 32 * kProducers, fresh);
     if (!ok && lane == 0 && a.status) atomicExch(a.status, (int)L3CI_ERR_DEVICE_WAIT);
     return;
   }
@@ -253,7 +287,7 @@ __global__ void __launch_bounds__(kScanThreads) recurrent_scan_kernel(const __gr
 #pragma unroll
         for (int j = 0; j < NR / 2; ++j) S2[c][j] = f2_fma(k2[j], u2, KIND == kDelta ? S2[c][j] : f2_mul(S2[c][j], g2[j]));
       }
-      if (!FUSE && l == 0 && live) {
+      if (l == 0 && live) {
 #pragma unroll
         for (int c = 0; c < C; ++c) out[c] = from_f32<S>(o[c]);
       }
@@ -280,24 +314,114 @@ __global__ void __launch_bounds__(kScanThreads) recurrent_scan_kernel(const __gr
       }
     }
   }
-  if (FUSE) {
-    // one token: the head's output is in this CTA (columns that do not exist are zeros)
-    float ss = 0.f;
+}
+
+// ---- one token ----------------------------------------------------------------------------------------------------
+constexpr int kStepThreads = 256;
+
+template <typename S, typename Q, int KIND, int RP>
+__global__ void __launch_bounds__(kStepThreads, RP <= 4 ? 5 : RP <= 8 ? 3 : 2) recurrent_step_kernel(const __grid_constant__ l3ci_recurrent_scan_args a) {
+  extern __shared__ __align__(16) float smem[];
+  __shared__ float red[32];
+  const int D = a.D, V = a.V, tid = threadIdx.x;
+  float *qs = smem, *ks = qs + D, *gs = ks + D;
+  float4* part = reinterpret_cast<float4*>(smem + (3 * D + 3) / 4 * 4);    // [2][groups][V / 4]
+  const int quads = V / 4, groups = kStepThreads / quads, quad = tid % quads, grp = tid / quads;
+  const int h = blockIdx.x % a.H, b = blockIdx.x / a.H, R = a.H / a.G;
+  const bool active = grp < groups;
+  pdl_wait();
+  pdl_launch_dependents();
+  const bool fresh = a.positions[b] == 0;
+  float4* state = reinterpret_cast<float4*>(a.state + b * a.state_sb + (long long)h * D * V) + quad;
+  float4 s[RP];
 #pragma unroll
-    for (int c = 0; c < C; ++c) ss = live ? fmaf(o[c], o[c], ss) : ss;
-    ss = group_sum<kWarp>(l == 0 ? ss : 0.f);
-    if (lane == 0) red[warp] = ss;
-    asm volatile("bar.sync 1, %0;" ::"r"(32 * p.consumers) : "memory");
-    ss = group_sum<kMaxConsumers>(lane % kMaxConsumers < p.consumers ? red[lane % kMaxConsumers] : 0.f);
-    const float inv = 1.f / sqrtf(ss / (float)V + a.eps);
-    if (l == 0 && live && ok) {
-      const S* gate = static_cast<const S*>(a.gate) + b * a.gate_st + h * a.gate_sh + c0;
-      S* dst = static_cast<S*>(a.out) + b * a.out_st + h * a.out_sh + c0;
+  for (int i = 0; i < RP; ++i) {
+    const int r = grp + i * groups;
+    s[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (active && !fresh && r < D) s[i] = __ldcs(state + (long long)r * quads);
+  }
+  const S* vp = static_cast<const S*>(a.v) + b * a.v_st + h * a.v_sh + 4 * quad;
+  const S* zp = static_cast<const S*>(a.gate) + b * a.gate_st + h * a.gate_sh + 4 * quad;
+  float v[4], z[4], w[4];
 #pragma unroll
-      for (int c = 0; c < C; ++c)
-        dst[c] = from_f32<S>(o[c] * inv * a.norm[h * a.norm_sh + c0 + c] * gate_value(to_f32(gate[c]), a.act));
+  for (int c = 0; c < 4; ++c) {
+    v[c] = to_f32(vp[c]);
+    z[c] = to_f32(zp[c]);
+    w[c] = a.norm[h * a.norm_sh + 4 * quad + c];
+  }
+  const float beta = KIND == kDelta ? a.beta[(long long)b * a.H + h] : 0.f;
+  float scalar = 0.f;
+  for (int d = tid; d < D; d += kStepThreads) {
+    const float q = to_f32(static_cast<const Q*>(a.q)[b * a.qk_st + (h / R) * a.qk_sh + d]);
+    const float k = to_f32(static_cast<const Q*>(a.k)[b * a.qk_st + (h / R) * a.qk_sh + d]);
+    float g = to_f32(static_cast<const Q*>(a.g)[b * a.g_st + h * a.g_sh + d]);
+    if (KIND == kTimeMix) {
+      g = expf(-expf(g + a.g_bias[h * D + d]));
+      scalar = fmaf(q * k, a.bonus[h * D + d], scalar);
+    } else {
+      scalar = fmaf(q, k, scalar);
+    }
+    qs[d] = q;
+    ks[d] = k;
+    gs[d] = g;
+  }
+  scalar = cta_sum(scalar, red, kStepThreads / kWarp);                     // (its barriers publish the vectors as well)
+  float4 ak = make_float4(0.f, 0.f, 0.f, 0.f), aq = ak;
+#pragma unroll
+  for (int i = 0; i < RP; ++i) {
+    const int r = grp + i * groups;
+    if (!active || r >= D) continue;
+    const float q = qs[r], g = gs[r];
+    if (KIND == kDelta) {
+      const float k = ks[r];
+      s[i].x *= g; s[i].y *= g; s[i].z *= g; s[i].w *= g;
+      ak.x = fmaf(s[i].x, k, ak.x); ak.y = fmaf(s[i].y, k, ak.y); ak.z = fmaf(s[i].z, k, ak.z); ak.w = fmaf(s[i].w, k, ak.w);
+    }
+    aq.x = fmaf(s[i].x, q, aq.x); aq.y = fmaf(s[i].y, q, aq.y); aq.z = fmaf(s[i].z, q, aq.z); aq.w = fmaf(s[i].w, q, aq.w);
+    if (KIND == kTimeMix) { s[i].x *= g; s[i].y *= g; s[i].z *= g; s[i].w *= g; }
+  }
+  if (active) {
+    if (KIND == kDelta) part[grp * quads + quad] = ak;
+    part[(groups + grp) * quads + quad] = aq;
+  }
+  __syncthreads();
+  float u[4] = {v[0], v[1], v[2], v[3]}, o[4] = {0.f, 0.f, 0.f, 0.f};
+  if (KIND == kDelta) {
+    float4 sum = make_float4(0.f, 0.f, 0.f, 0.f);
+    for (int i = 0; i < groups; ++i) {
+      const float4 x = part[i * quads + quad];
+      sum.x += x.x; sum.y += x.y; sum.z += x.z; sum.w += x.w;
+    }
+    u[0] = beta * (v[0] - sum.x); u[1] = beta * (v[1] - sum.y); u[2] = beta * (v[2] - sum.z); u[3] = beta * (v[3] - sum.w);
+  }
+#pragma unroll
+  for (int i = 0; i < RP; ++i) {
+    const int r = grp + i * groups;
+    if (!active || r >= D) continue;
+    const float k = ks[r];
+    s[i].x = fmaf(k, u[0], s[i].x); s[i].y = fmaf(k, u[1], s[i].y); s[i].z = fmaf(k, u[2], s[i].z); s[i].w = fmaf(k, u[3], s[i].w);
+    __stcs(state + (long long)r * quads, s[i]);
+  }
+  float ss = 0.f;
+  if (grp == 0) {
+    for (int i = 0; i < groups; ++i) {
+      const float4 x = part[(groups + i) * quads + quad];
+      o[0] += x.x; o[1] += x.y; o[2] += x.z; o[3] += x.w;
+    }
+#pragma unroll
+    for (int c = 0; c < 4; ++c) {
+      o[c] = fmaf(scalar, u[c], o[c]);
+      ss = fmaf(o[c], o[c], ss);
     }
   }
+  ss = cta_sum(ss, red, kStepThreads / kWarp);
+  if (grp == 0) {
+    const float inv = 1.f / sqrtf(ss / (float)V + a.eps);
+    S* dst = static_cast<S*>(a.out) + b * a.out_st + h * a.out_sh + 4 * quad;
+#pragma unroll
+    for (int c = 0; c < 4; ++c) dst[c] = from_f32<S>(o[c] * inv * w[c] * gate_value(z[c], a.act));
+  }
+  if (a.tail) move_tails<S>(a, b, h, tid, kStepThreads, fresh);
 }
 
 // out[row, h, :] <- out / rms(out) * norm * act(gate), in place: a warp per (row, head)
@@ -355,9 +479,11 @@ head_norm_gate_kernel(S* __restrict__ out, long long out_st, long long out_sh, c
 }
 
 // ---- inputs of the delta rule -----------------------------------------------------------------------------------
-constexpr int kRun = 4;            // consecutive tokens of a warp
+constexpr int kRun = 8;            // consecutive tokens of a warp
+constexpr int kMaxTaps = 4;        // taps whose inputs stay in registers along the run
 
-template <typename S, int VEC>
+// TAPS > 0: the run's inputs are all asked for at once and every one is loaded once; 0: any number of taps.
+template <typename S, int VEC, int TAPS>
 __global__ void __launch_bounds__(256) delta_inputs_kernel(const l3ci_delta_inputs_args a, int runs, long long tasks) {
   pdl_wait();
   pdl_launch_dependents();
@@ -375,22 +501,26 @@ __global__ void __launch_bounds__(256) delta_inputs_kernel(const l3ci_delta_inpu
   if (what >= 2 * a.G + a.H) {
     const int h = what - 2 * a.G - a.H;
     const float rate = expf(a.a_log[h]);
-    for (int x = 0; x < n; ++x) {
-      const long long row = row0 + t0 + x;
-      const S* src = static_cast<const S*>(a.a) + row * a.a_st + (long long)h * a.D;
-      for (int c = lane * VEC; c < a.D; c += 32 * VEC) {
-        float z[VEC], bias[VEC];
-        load_vec<S, VEC>(src + c, z);
-        load_vec<float, VEC>(a.dt_bias + (long long)h * a.D + c, bias);
+    const S* src = static_cast<const S*>(a.a) + (row0 + t0) * a.a_st + (long long)h * a.D;
+    if (lane < n) {
+      const float z = to_f32(static_cast<const S*>(a.b)[(row0 + t0 + lane) * a.b_st + h]);
+      a.beta_out[(row0 + t0 + lane) * a.H + h] = sigmoid(z);
+    }
+    for (int c = lane * VEC; c < a.D; c += 32 * VEC) {
+      float z[kRun][VEC], bias[VEC];
+      load_vec<float, VEC>(a.dt_bias + (long long)h * a.D + c, bias);
+#pragma unroll
+      for (int x = 0; x < kRun; ++x) load_vec<S, VEC>(src + min(x, n - 1) * a.a_st + c, z[x]);
+#pragma unroll
+      for (int x = 0; x < kRun; ++x) {
+        if (x >= n) break;
 #pragma unroll
         for (int k = 0; k < VEC; ++k) {
-          const float y = z[k] + bias[k];
-          const float sp = fmaxf(y, 0.f) + log1pf(expf(-fabsf(y)));
-          z[k] = expf(-rate * sp);
+          const float y = z[x][k] + bias[k];
+          z[x][k] = expf(-rate * (fmaxf(y, 0.f) + log1pf(expf(-fabsf(y)))));
         }
-        store_vec<float, VEC>(a.decay_out + (row * a.H + h) * a.D + c, z);
+        store_vec<float, VEC>(a.decay_out + ((row0 + t0 + x) * a.H + h) * a.D + c, z[x]);
       }
-      if (lane == 0) a.beta_out[row * a.H + h] = sigmoid(to_f32(static_cast<const S*>(a.b)[row * a.b_st + h]));
     }
     return;
   }
@@ -400,33 +530,81 @@ __global__ void __launch_bounds__(256) delta_inputs_kernel(const l3ci_delta_inpu
   const bool fresh = a.positions[b] == 0;
   const S* in = static_cast<const S*>(a.p) + row0 * a.p_st + ch0;
   const S* tail = static_cast<const S*>(a.tail) + b * a.tail_sb + ch0;
+  const int taps = TAPS > 0 ? TAPS : a.taps;
+  constexpr int kKeep = VEC >= 4 ? 2 : 8;      // 256 channels
+  auto activation = [](float z) {
+    if constexpr (sizeof(S) == 4) return z * sigmoid(z);
+    else return __fdividef(z, 1.f + __expf(-z));   // (bf16 models: rounded to bf16, or made a unit vector, right after)
+  };
+  // input of the sequence's token t (of this call; before it: the carried ones) at channel c
+  auto input = [&](int t, int c, float (&f)[VEC]) {
+    if (t >= 0) {
+      load_vec<S, VEC>(in + (long long)t * a.p_st + c, f);
+    } else {
+#pragma unroll
+      for (int k = 0; k < VEC; ++k) f[k] = 0.f;
+      if (!fresh) load_vec<S, VEC>(tail + (taps - 1 + t) * C_all + c, f);
+    }
+  };
+  auto store = [&](int x, int c, const float (&y)[VEC], float f) {
+    float r[VEC];
+#pragma unroll
+    for (int k = 0; k < VEC; ++k) r[k] = y[k] * f;
+    const long long row = row0 + t0 + x;
+    if (is_v) store_vec<S, VEC>(static_cast<S*>(a.v_out) + row * a.H * a.V + (long long)(what - 2 * a.G) * a.V + c, r);
+    else store_vec<float, VEC>(a.qk_out + row * 2 * GD + ch0 + c, r);
+  };
+  auto unit = [&](float ss) { return is_v ? 1.f : 1.f / sqrtf(ss + a.unit_eps) / (what < a.G ? sqrtf((float)a.D) : 1.f); };
+  if (TAPS > 0 && (is_v || size <= 32 * VEC)) {
+    constexpr int kTaps = TAPS > 0 ? TAPS : 1;
+    for (int c = lane * VEC; c < (is_v ? size : 32 * VEC); c += 32 * VEC) {    // (every lane takes part in a unit vector's sums)
+      const bool mine = c < size;
+      const int at = mine ? c : 0;
+      float f[kRun + kTaps - 1][VEC], w[kTaps][VEC];
+#pragma unroll
+      for (int i = 0; i < kRun + kTaps - 1; ++i) input(min(t0 - (kTaps - 1) + i, a.T - 1), at, f[i]);
+#pragma unroll
+      for (int i = 0; i < kTaps; ++i) load_vec<float, VEC>(a.conv + i * C_all + ch0 + at, w[i]);
+#pragma unroll
+      for (int x = 0; x < kRun; ++x) {
+        if (x >= n) break;
+        float y[VEC], ss = 0.f;
+#pragma unroll
+        for (int k = 0; k < VEC; ++k) {
+          y[k] = 0.f;
+#pragma unroll
+          for (int i = 0; i < kTaps; ++i) y[k] = fmaf(f[x + i][k], w[i][k], y[k]);
+          y[k] = activation(y[k]);
+          ss = mine ? fmaf(y[k], y[k], ss) : ss;
+        }
+        if (!is_v) ss = group_sum<kWarp>(ss);
+        if (mine) store(x, c, y, unit(ss));
+      }
+    }
+    return;
+  }
   for (int x = 0; x < n; ++x) {
-    const int t = t0 + x;
-    const long long row = row0 + t;
     auto convolve = [&](int c, float (&y)[VEC]) {
 #pragma unroll
       for (int k = 0; k < VEC; ++k) y[k] = 0.f;
-      for (int i = 0; i < a.taps; ++i) {
-        const int at = t - (a.taps - 1) + i;
-        if (at < 0 && fresh) continue;
+      for (int i = 0; i < taps; ++i) {
         float f[VEC], w[VEC];
-        load_vec<S, VEC>(at >= 0 ? in + (long long)at * a.p_st + c : tail + (a.taps - 1 + at) * C_all + c, f);
+        input(t0 + x - (taps - 1) + i, c, f);
         load_vec<float, VEC>(a.conv + i * C_all + ch0 + c, w);
 #pragma unroll
         for (int k = 0; k < VEC; ++k) y[k] = fmaf(f[k], w[k], y[k]);
       }
 #pragma unroll
-      for (int k = 0; k < VEC; ++k) y[k] *= sigmoid(y[k]);
+      for (int k = 0; k < VEC; ++k) y[k] = activation(y[k]);
     };
     if (is_v) {
       for (int c = lane * VEC; c < size; c += 32 * VEC) {
         float y[VEC];
         convolve(c, y);
-        store_vec<S, VEC>(static_cast<S*>(a.v_out) + row * a.H * a.V + (long long)(what - 2 * a.G) * a.V + c, y);
+        store(x, c, y, 1.f);
       }
       continue;
     }
-    constexpr int kKeep = VEC >= 4 ? 2 : 8;    // 256 channels
     float y[kKeep][VEC], ss = 0.f;
 #pragma unroll
     for (int i = 0; i < kKeep; ++i) {
@@ -437,16 +615,11 @@ __global__ void __launch_bounds__(256) delta_inputs_kernel(const l3ci_delta_inpu
         for (int k = 0; k < VEC; ++k) ss = fmaf(y[i][k], y[i][k], ss);
       }
     }
-    float f = 1.f / sqrtf(group_sum<kWarp>(ss) + a.unit_eps);
-    if (what < a.G) f /= sqrtf((float)a.D);
+    const float f = unit(group_sum<kWarp>(ss));
 #pragma unroll
     for (int i = 0; i < kKeep; ++i) {
       const int c = (i * 32 + lane) * VEC;
-      if (c < size) {
-#pragma unroll
-        for (int k = 0; k < VEC; ++k) y[i][k] *= f;
-        store_vec<float, VEC>(a.qk_out + row * 2 * GD + ch0 + c, y[i]);
-      }
+      if (c < size) store(x, c, y[i], f);
     }
   }
 }
@@ -455,51 +628,62 @@ constexpr int kMaxD = 256;         // key channels of a head
 
 template <typename S, typename Q, int KIND, int NR, int C>
 int launch_scan(const ScanParams& p, cudaStream_t stream) {
-  const size_t smem = (size_t)kRing * kChunk * (3 * NR * 8 + p.cols + 2) * 4 + kMaxConsumers * 4 + 2 * kRing * 8;
-  const dim3 grid((unsigned)((long long)p.a.B * p.a.H * p.splits)), block(32 * (p.consumers + kProducers));
-  static bool configured[2][64] = {};
-  auto go = [&](auto kernel, int which) -> int {
-    int dev = 0;
-    L3CI_CUDA_TRY(cudaGetDevice(&dev));
-    if (smem > (48 << 10) && (dev < 0 || dev >= 64 || !configured[which][dev])) {
-      L3CI_CUDA_TRY(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, max_smem_optin()));
-      if (dev >= 0 && dev < 64) configured[which][dev] = true;
-    }
-    L3CI_LAUNCH("recurrent_scan_kernel", kernel, grid, block, smem, stream, p);
+  const size_t smem = (size_t)kRing * kChunk * (3 * NR * 8 + p.cols + 2) * 4 + 2 * kRing * 8;
+  static bool configured[64] = {false};
+  int dev = 0;
+  L3CI_CUDA_TRY(cudaGetDevice(&dev));
+  if (smem > (48 << 10) && (dev < 0 || dev >= 64 || !configured[dev])) {
+    L3CI_CUDA_TRY(cudaFuncSetAttribute(recurrent_scan_kernel<S, Q, KIND, NR, C>, cudaFuncAttributeMaxDynamicSharedMemorySize, max_smem_optin()));
+    if (dev >= 0 && dev < 64) configured[dev] = true;
+  }
+  L3CI_LAUNCH("recurrent_scan_kernel", recurrent_scan_kernel<S, Q, KIND, NR, C>, dim3((unsigned)((long long)p.a.B * p.a.H * p.splits)),
+              dim3(32 * (p.consumers + kProducers)), smem, stream, p);
+  return L3CI_OK;
+}
+
+// One token per sequence, if its sizes suit: rows of whole 16-byte vectors, at most 16 of them per thread.
+template <typename S, typename Q, int KIND>
+bool step_applies(const l3ci_recurrent_scan_args* a) {
+  if (a->T != 1 || a->V % 4 || a->V > 4 * kStepThreads || a->state_sb % 4 || !aligned16(a->state)) return false;
+  const int groups = kStepThreads / (a->V / 4);
+  return (a->D + groups - 1) / groups <= 16;
+}
+template <typename S, typename Q, int KIND>
+int step_launch(const l3ci_recurrent_scan_args* a, cudaStream_t stream) {
+  const int quads = a->V / 4, groups = kStepThreads / quads, rows = (a->D + groups - 1) / groups;
+  const size_t smem = sizeof(float) * ((3 * a->D + 3) / 4 * 4 + 2 * (size_t)groups * a->V);
+  const long long ctas = (long long)a->B * a->H;
+  if (ctas > 0x7fffffffLL) return fail(L3CI_ERR_INVALID, "recurrent_scan: too many sequences");
+  auto go = [&](auto kernel) -> int {
+    L3CI_LAUNCH("recurrent_step_kernel", kernel, dim3((unsigned)ctas), dim3(kStepThreads), smem, stream, *a);
     return L3CI_OK;
   };
-  if (p.a.T == 1 && p.splits == 1) return go(recurrent_scan_kernel<S, Q, KIND, NR, C, true>, 1);
-  return go(recurrent_scan_kernel<S, Q, KIND, NR, C, false>, 0);
+  return rows <= 4 ? go(recurrent_step_kernel<S, Q, KIND, 4>) : rows <= 8 ? go(recurrent_step_kernel<S, Q, KIND, 8>)
+                                                                         : go(recurrent_step_kernel<S, Q, KIND, 16>);
 }
 
 template <typename S, typename Q, int KIND>
 int scan_typed(const l3ci_recurrent_scan_args* a, cudaStream_t stream) {
+  if (step_applies<S, Q, KIND>(a)) return step_launch<S, Q, KIND>(a, stream);
   ScanParams p = {};
   p.a = *a;
   const long long heads = (long long)a->B * a->H;
   const int sms = sm_count() > 0 ? sm_count() : 148;
-  // columns per thread: as many as one CTA per head allows for a single token (wide accesses of the state), else what leaves
-  // enough CTAs for the device
+  // columns per thread: as many as leave enough CTAs for the device
   const int widest = a->V % 4 == 0 && a->state_sb % 4 == 0 && (reinterpret_cast<uintptr_t>(a->state) & 15) == 0   ? 4
                      : a->V % 2 == 0 && a->state_sb % 2 == 0 && (reinterpret_cast<uintptr_t>(a->state) & 7) == 0 ? 2
                                                                                                                  : 1;
-  int C = widest;
-  if (a->T == 1) {
-    const int per = 4 * C * kMaxConsumers;
-    p.splits = (a->V + per - 1) / per;
-    p.consumers = ((a->V + p.splits - 1) / p.splits + 4 * C - 1) / (4 * C);
-  } else {
-    const struct { int C, W; } shapes[] = {{4, 8}, {2, 8}, {2, 4}, {1, 4}, {1, 2}};
-    for (const auto& s : shapes) {
-      if (s.C > widest && s.C > 1) continue;
-      C = s.C;
-      p.consumers = s.W;
-      p.splits = (a->V + 4 * C * s.W - 1) / (4 * C * s.W);
-      if (heads * p.splits * 5 >= 4LL * sms) break;
-    }
-    const int need = (a->V + 4 * C - 1) / (4 * C);
-    if (p.consumers > need) p.consumers = need;
+  int C = 1;
+  const struct { int C, W; } shapes[] = {{4, 8}, {2, 8}, {2, 4}, {1, 4}, {1, 2}};
+  for (const auto& s : shapes) {
+    if (s.C > widest && s.C > 1) continue;
+    C = s.C;
+    p.consumers = s.W;
+    p.splits = (a->V + 4 * C * s.W - 1) / (4 * C * s.W);
+    if (heads * p.splits * 5 >= 4LL * sms) break;
   }
+  const int need = (a->V + 4 * C - 1) / (4 * C);
+  if (p.consumers > need) p.consumers = need;
   p.cols = 4 * C * p.consumers;
   if (p.splits * (long long)p.cols < a->V) p.splits = (a->V + p.cols - 1) / p.cols;
   if (heads * p.splits > 0x7fffffffLL) return fail(L3CI_ERR_INVALID, "recurrent_scan: too many sequences");
@@ -518,7 +702,7 @@ int scan_typed(const l3ci_recurrent_scan_args* a, cudaStream_t stream) {
   if (C == 4) st = rows(std::integral_constant<int, 4>{});
   else if (C == 2) st = rows(std::integral_constant<int, 2>{});
   else st = rows(std::integral_constant<int, 1>{});
-  if (st || (a->T == 1 && p.splits == 1)) return st;
+  if (st) return st;
   // norm and gate of the rows the scan has written
   const long long units = heads * a->T;
   if ((units + 7) / 8 > 0x7fffffffLL) return fail(L3CI_ERR_INVALID, "recurrent_scan: too many rows");
@@ -564,7 +748,14 @@ int l3ci_delta_inputs(const l3ci_delta_inputs_args* a) {
       L3CI_LAUNCH("delta_inputs_kernel", kernel, dim3((unsigned)((tasks + 7) / 8)), dim3(256), 0, s, *a, runs, tasks);
       return L3CI_OK;
     };
-    return v4 ? go(delta_inputs_kernel<S, 4>) : go(delta_inputs_kernel<S, 1>);
+    if (!v4) return go(delta_inputs_kernel<S, 1, 0>);
+    switch (a->taps) {
+      case 1: return go(delta_inputs_kernel<S, 4, 1>);
+      case 2: return go(delta_inputs_kernel<S, 4, 2>);
+      case 3: return go(delta_inputs_kernel<S, 4, 3>);
+      case kMaxTaps: return go(delta_inputs_kernel<S, 4, kMaxTaps>);
+    }
+    return go(delta_inputs_kernel<S, 4, 0>);
   };
   return a->dtype == L3CI_BF16 ? typed(__nv_bfloat16{}) : typed(float{});
 }

@@ -21,6 +21,7 @@ namespace l3ci {
 namespace {
 
 constexpr int kMaxWarps = 16;
+constexpr int kManyVpt = 8;    // vectors of a thread when there are many rows
 
 // Mean and 1 / sqrt(variance + eps) of a row of `width` values; the thread's values are the first `valid` of v.
 template <int N>
@@ -30,7 +31,7 @@ __device__ __forceinline__ void row_stats(const float (&v)[N], int valid, int wi
 #pragma unroll
   for (int i = 0; i < N; ++i)
     if (i < valid) s += v[i];
-  const float cnt = (float)__reduce_add_sync(kFullMask, valid);
+  const float cnt = warps > 1 ? (float)__reduce_add_sync(kFullMask, valid) : (float)width;
   mean = cnt > 0.f ? group_sum<kWarp>(s) / cnt : 0.f;
   float m2 = 0.f;
 #pragma unroll
@@ -59,7 +60,7 @@ __device__ __forceinline__ float sinusoid(int p, double freq, bool cosine) {
 }
 
 template <typename S, int VEC, int VPT>
-__global__ void __launch_bounds__(512) residual_norm_kernel(const l3ci_residual_norm_args a) {
+__global__ void __launch_bounds__(VPT >= 16 ? 256 : 512) residual_norm_kernel(const l3ci_residual_norm_args a) {
   __shared__ float sm[2][kMaxWarps][3];
   const int tid = threadIdx.x, width = (int)a.width;
   int col[VPT], chunks = 0;
@@ -185,15 +186,13 @@ int residual_norm_typed(const l3ci_residual_norm_args* a) {
                   ok(a->step, 16) && ok(a->pre_w, 16) && ok(a->pre_b, 16) && ok(a->out, s4) && a->out_stride % 4 == 0 && ok(a->table, s4) &&
                   ok(a->x0, s4) && a->x0_stride % 4 == 0;
   const long long units = v4 ? a->width / 4 : a->width;
-  // few rows: as many threads as there are vectors; many rows: more vectors a thread, more CTAs on an SM
-  const int most = a->rows > 2LL * (sm_count() > 0 ? sm_count() : 148) ? 256 : 512;
-  int threads = 32;
-  while (threads < most && threads < units) threads *= 2;
-  int vpt = 1;
-  while ((long long)vpt * threads < units) {
-    if (vpt >= 4 && threads < 512) threads *= 2;
-    else vpt *= 2;
-  }
+  // few rows: as many threads as there are vectors; many rows: few threads with many vectors each, so that little of the work
+  // is reductions and many rows are on an SM
+  const bool many = a->rows > 4LL * (sm_count() > 0 ? sm_count() : 148);
+  int threads = 32, vpt = 1;
+  while ((many && v4 ? kManyVpt : 1) * threads < units && threads < 512) threads *= 2;
+  while ((long long)vpt * threads < units) vpt *= 2;
+  if (threads > (vpt >= 16 ? 256 : 512)) return fail(L3CI_ERR_UNSUPPORTED, "residual_norm: width %lld", (long long)a->width);
   auto go = [&](auto kernel) -> int {
     L3CI_LAUNCH("residual_norm_kernel", kernel, dim3((unsigned)a->rows), dim3(threads), 0, reinterpret_cast<cudaStream_t>(a->stream), *a);
     return L3CI_OK;
@@ -204,6 +203,7 @@ int residual_norm_typed(const l3ci_residual_norm_args* a) {
       case 2: return go(residual_norm_kernel<S, 4, 2>);
       case 4: return go(residual_norm_kernel<S, 4, 4>);
       case 8: return go(residual_norm_kernel<S, 4, 8>);
+      case 16: return go(residual_norm_kernel<S, 4, 16>);
     }
   } else {
     switch (vpt) {

@@ -28,6 +28,16 @@ __device__ __forceinline__ float gated_activation(float z, float u, float limit,
   return z / (1.f + expf(-z)) * u;
 }
 
+// The same to bf16 accuracy (relative error about 1e-6), without the divide's branches.
+__device__ __forceinline__ float gated_activation_fast(float z, float u, float limit, float alpha) {
+  if (limit > 0.f) {
+    z = fminf(z, limit);
+    u = fminf(fmaxf(u, -limit), limit) + 1.f;
+    return __fdividef(z, 1.f + __expf(-alpha * z)) * u;
+  }
+  return __fdividef(z, 1.f + __expf(-z)) * u;
+}
+
 template <int BYTES>
 struct Raw;
 template <>

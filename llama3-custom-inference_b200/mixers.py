@@ -103,7 +103,7 @@ def load() -> C.CDLL:
     lib.l3ci_token_shift.argtypes = [vp, vp, vp, i64, vp, vp, i32, i32, i32, i64, i32, vp]
     lib.l3ci_delta_inputs.argtypes = [C.POINTER(DeltaInputsArgs)]
     lib.l3ci_recurrent_scan.argtypes = [C.POINTER(RecurrentScanArgs)]
-    lib.l3ci_moe_route.argtypes = [vp, vp, vp, vp, vp, vp, vp, i64, i64, i32, i32, i32, vp]
+    lib.l3ci_moe_route.argtypes = [vp, vp, vp, vp, vp, vp, i64, i32, i32, vp]
     lib.l3ci_moe_gather.argtypes = [vp, vp, vp, vp, vp, vp, i64, i64, i32, i32, i32, vp]
     lib.l3ci_moe_gemm.argtypes = [C.POINTER(MoeGemmArgs)]
     lib.l3ci_moe_gemm_variant.argtypes = [C.POINTER(MoeGemmArgs)]
@@ -322,18 +322,17 @@ def recurrent_scan(q, k, v, g, state, positions, norm, gate, *, act: int, eps: f
     return out.view(B, T, H * V)
 
 
-def moe_route(h, router, bias, top: int):
-    """h [rows, width], router [experts, width] -> experts, ranks (int32 [rows, top]), weights [rows, top], counts [experts]."""
-    _cuda(h, router)
-    rows, E = h.shape[0], router.shape[0]
-    assert h.is_contiguous() and router.is_contiguous() and router.dtype == h.dtype and bias.dtype == torch.float32
-    i32 = dict(dtype=torch.int32, device=h.device)
+def moe_route(logits, bias, top: int):
+    """logits fp32 [rows, experts] -> experts, ranks (int32 [rows, top]), weights [rows, top], counts [experts]."""
+    _cuda(logits, bias)
+    rows, E = logits.shape
+    assert logits.is_contiguous() and logits.dtype == bias.dtype == torch.float32
+    i32 = dict(dtype=torch.int32, device=logits.device)
     experts, ranks, counts = torch.empty(rows, top, **i32), torch.empty(rows, top, **i32), torch.empty(E, **i32)
-    weights = torch.empty(rows, top, dtype=torch.float32, device=h.device)
-    with _on(h):
-        _check(load().l3ci_moe_route(h.data_ptr(), router.data_ptr(), bias.data_ptr(), experts.data_ptr(), ranks.data_ptr(),
-                                     weights.data_ptr(), counts.data_ptr(), rows, h.shape[1], E, top, DTYPE_CODES[h.dtype], _stream(h)),
-               "l3ci_moe_route")
+    weights = torch.empty(rows, top, dtype=torch.float32, device=logits.device)
+    with _on(logits):
+        _check(load().l3ci_moe_route(logits.data_ptr(), bias.data_ptr(), experts.data_ptr(), ranks.data_ptr(), weights.data_ptr(),
+                                     counts.data_ptr(), rows, E, top, _stream(logits)), "l3ci_moe_route")
     return experts, ranks, weights, counts
 
 

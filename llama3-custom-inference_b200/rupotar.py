@@ -353,17 +353,14 @@ class RupotarDecoder(DecodeLoop):
         if isinstance(ff, Dense):
             return {"y": F.linear(mixers.gated_act(F.linear(h, w.gate_up)), w.down)}
         rows = h.view(-1, h.shape[-1])
-        experts, ranks, weights, counts = mixers.moe_route(rows, w.router, w.router_b, ff.top)
+        experts, ranks, weights, counts = mixers.moe_route(self._product32(rows, w.router), w.router_b, ff.top)
         x, part_rows = mixers.moe_gather(rows, experts, ranks, counts)
         a = mixers.moe_gemm(x, w.gate_up, counts, limit=ff.limit, alpha=EXPERT_ALPHA)
         return {"y": mixers.moe_gemm(a, w.down, counts), "part_rows": part_rows, "part_weights": weights}
 
-    def _loop_product(self, cat):
-        """W_in [x; embedding output] in fp32: it becomes the residual stream."""
-        flat = cat.view(-1, cat.shape[-1])
-        if self.dtype == torch.float32:
-            return torch.mm(flat, self.loop_in.t())
-        return torch.mm(flat, self.loop_in.t(), out_dtype=torch.float32)
+    def _product32(self, x, w):
+        """x w^T in fp32: products of two bf16 numbers are exact, the sum is not rounded to bf16."""
+        return torch.mm(x, w.t()) if x.dtype == torch.float32 else torch.mm(x, w.t(), out_dtype=torch.float32)
 
     # ---- one forward pass over T new tokens per sequence ------------------------------------------------------
     def forward(self, tokens: torch.Tensor, positions: torch.Tensor, seq_lens: torch.Tensor, start_pos: int = 0,
@@ -394,7 +391,7 @@ class RupotarDecoder(DecodeLoop):
                 mix = self._attention if isinstance(m, Attention) else self._channel_delta if isinstance(m, ChannelDelta) else self._wkv
                 with nvtx_range("layer"):
                     if run.step is not None:
-                        h = mixers.residual_norm(self._loop_product(cat), x, dtype=self.dtype, reset=True, step=self.loop_step[run.step],
+                        h = mixers.residual_norm(self._product32(cat.view(B * T, 2 * E), self.loop_in), x, dtype=self.dtype, reset=True, step=self.loop_step[run.step],
                                                  pre=w.norm1, eps=eps)
                     added, post = {"y": F.linear(mix(m, w, planes, h, positions, start_pos), w.o)}, w.norm1b
                     if ff is not None:

@@ -309,10 +309,9 @@ def test_scan_of_sequences_at_different_places(pkg, device):
 
 # ---- experts ----------------------------------------------------------------------------------------------------
 def route(pkg, device, rows, width, E, top, dtype, seed=0, skew=0.0):
-    h, router, bias = rand(rows, width, seed=seed, dtype=dtype), rand(E, width, seed=seed + 1, dtype=dtype), rand(E, seed=seed + 2, dtype=F32)
+    h, logits, bias = rand(rows, width, seed=seed, dtype=dtype), rand(rows, E, seed=seed + 1, scale=5, dtype=F32), rand(E, seed=seed + 2, dtype=F32)
     bias[0] += skew
-    z = h.double() @ router.double().T + bias.double()
-    return h, z, pkg.mixers.moe_route(h.to(device), router.to(device), bias.to(device), top)
+    return h, logits.double() + bias.double(), pkg.mixers.moe_route(logits.to(device), bias.to(device), top)
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
@@ -324,7 +323,7 @@ def test_routing_and_sorting(pkg, device, dtype, rows, width, E, top, skew):
     clear = torch.ones(rows, dtype=torch.bool)
     if top < E:
         s = z.sort(dim=-1, descending=True).values
-        clear = s[:, top - 1] - s[:, top] > 1e-3
+        clear = s[:, top - 1] - s[:, top] > 1e-5
     e = experts.cpu().long()
     assert torch.equal(e.sort(-1).values[clear], chosen.sort(-1).values[clear]) and clear.float().mean() > 0.9
     assert (weights.cpu().double() - w)[clear].abs().max() < 2e-4
@@ -336,6 +335,15 @@ def test_routing_and_sorting(pkg, device, dtype, rows, width, E, top, skew):
     by_place[at_] = e.flatten()
     assert (by_place.diff() >= 0).all()                                                           # expert by expert
     assert torch.equal(x.cpu()[at_], h.repeat_interleave(top, 0))
+
+
+def test_equal_logits_take_the_smaller_index(pkg, device):
+    for E in (5, 33, 100):
+        experts, _, weights, _ = pkg.mixers.moe_route(torch.zeros(40, E, device=device), torch.zeros(E, device=device), 3)
+        assert (experts.cpu() == torch.arange(3)).all() and (weights - 1 / 3).abs().max() < 1e-6
+    z = torch.full((40, 50), -1e30, device=device)
+    z[:, 41], z[:, 7], z[:, 20] = float("inf"), float("nan"), -5.0
+    assert (pkg.mixers.moe_route(z, torch.zeros(50, device=device), 3)[0].cpu() == torch.tensor([41, 20, 0])).all()
 
 
 @pytest.mark.parametrize("E,counts_kind", [(4, "even"), (7, "one"), (40, "random")])

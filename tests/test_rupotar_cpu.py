@@ -101,8 +101,8 @@ def test_argument_validation_happens_before_cuda(pkg):
     assert lib.l3ci_residual_norm(C.byref(r)) == bad
     r = m.ResidualNormArgs(x=fake, rows=2, width=8, y=fake, parts=0)
     assert lib.l3ci_residual_norm(C.byref(r)) == bad
-    assert lib.l3ci_moe_route(fake, fake, fake, fake, fake, fake, fake, 4, 8, 3, 4, 0, None) == bad       # four of three experts
-    assert lib.l3ci_moe_route(fake, fake, fake, fake, fake, fake, fake, 4, 8, 5000, 4, 0, None) == bad
+    assert lib.l3ci_moe_route(fake, fake, fake, fake, fake, fake, 4, 3, 4, None) == bad       # four of three experts
+    assert lib.l3ci_moe_route(fake, fake, fake, fake, fake, fake, 4, 5000, 4, None) == bad
     assert lib.l3ci_moe_gather(fake, fake, fake, fake, fake, fake, 0, 8, 4, 2, 0, None) == ok
     g = m.MoeGemmArgs(x=fake, w=fake, out=fake, counts=fake, rows=4, K=12, N=8, n_experts=2, variant=2)
     assert lib.l3ci_moe_gemm_variant(C.byref(g)) == -1 and lib.l3ci_moe_gemm(C.byref(g)) == unsupported     # rows of 24 bytes
