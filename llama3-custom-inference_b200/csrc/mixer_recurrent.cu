@@ -1,22 +1,25 @@
 // Linear recurrences over a matrix state per (sequence, head), fp32: the gated delta rule with a decay per key channel, and
 // time mixing with a bonus for the current token (include/l3ci_mixers.h).
 //
-// recurrent_scan_kernel.  The columns of the state do not depend on one another, so a CTA takes a run of columns of one head
-// through all tokens of the call.  The state lives in registers: 8 lanes share C columns, a lane holds NR of their rows (rows
-// 4 l .. 4 l + 3 of every 32, so that the 8 lanes' 16-byte reads of a token's q, k, g cover 128 bytes of shared memory).  Both
-// products of the delta rule are taken over the decayed state in one pass,
-//     S^T k  and  S^T q,   u = beta (v - S^T k),   o = S^T q + (k . q) u,
-// so that a token costs one reduction over the 8 lanes; k . q (and the bonus product of time mixing) is the same for all
-// columns and comes with the token.  Rows go two at a time through packed fp32 instructions.
-// Four producer warps stage the next tokens (convert, form decays, take the scalar products) in a ring of two chunks while
-// the others compute; a chunk's loads are all in flight before the chunk ahead of it is handed over.  The head's output norm
-// and gate follow in a pass over the output rows (head_norm_gate_kernel).
+// recurrent_scan_kernel: several tokens.  The columns of the state do not depend on one another, so a warp takes C columns of one
+// head through all tokens of the call, the state in its registers: a lane holds NR rows of the C columns, rows two at a time
+// through packed fp32 instructions.  What the tokens bring (q, k, g, v) is the same for all columns of a head; it comes
+// through a ring of stages of 16 tokens in shared memory, filled by bulk tensor copies.
+//   The delta rule's chain runs through S^T k, a sum over all rows.  With S'_t = g_t S_{t-1} (decayed, not yet written to),
+//       S'_t^T k_t = (g_t k_t)^T S'_{t-1} + ((g_t k_t) . k_{t-1}) u_{t-1},
+//   so the sum over the state that token t needs is taken of S'_{t-1}, before u_{t-1} is known, and only two
+//   multiply-adds follow u_{t-1} on the way to u_t.  The scalar (g_t k_t) . k_{t-1} is the same for all columns: a helper
+//   warp forms it.  Outputs are not on the chain: the lanes' shares of 32 of them (32 / C tokens of C
+//   columns) meet in a patch of shared memory of the warp, after which a lane holds one output.
+//   Time mixing has no chain through the sums; its helper warps form the decays.
+// The head's output norm and gate follow in a pass over the output rows (head_norm_gate_kernel).
 //
 // recurrent_step_kernel: one token.  A CTA per head streams the state through registers, four columns and every n-th row a
 // thread (whole rows per warp access), meets in shared memory for the two products, and applies norm and gate itself.
 //
 // delta_inputs_kernel: convolution, activation, unit norms, step sizes and decays of all tokens at once; a warp per run of
 // tokens and head of one of q, k, v or the decay.
+#include <cuda.h>
 #include <cuda_bf16.h>
 #include <cuda_runtime.h>
 #include <math.h>
@@ -26,6 +29,7 @@
 #include "mixer_types.cuh"
 #include "ptx_sm100.cuh"
 #include "tcgen05.cuh"
+#include "tensor_map.h"
 #include "warp_reduce.cuh"
 
 namespace l3ci {
@@ -33,11 +37,14 @@ namespace {
 
 constexpr int kDelta = 0, kTimeMix = 1;
 constexpr int kChunk = 16;         // tokens per stage
-constexpr int kRing = 2;           // stages
-constexpr int kProducers = 4;      // warps
-constexpr int kPerProducer = kChunk / kProducers;
-constexpr int kMaxConsumers = 8;   // warps
-constexpr int kScanThreads = 32 * (kMaxConsumers + kProducers);
+constexpr int kMaxRing = 4;        // stages
+constexpr int kMaxConsumers[2] = {8, 16};   // warps, by kind
+constexpr int kHelpers[2] = {1, 2};   // warps, by kind
+// A warp's patch of output shares: 32 / C tokens of 32 lanes of C floats, tokens a little apart (no bank conflicts).
+template <int C>
+constexpr int kPatchToken = 32 * C + (C == 4 ? 16 : 32);   // floats
+constexpr int kPatchBytes = 8 * kPatchToken<4> * 4;
+static_assert(kPatchBytes >= 4 * kPatchToken<8> * 4, "a patch holds either form");
 
 __device__ __forceinline__ float sigmoid(float z) { return 1.f / (1.f + expf(-z)); }
 __device__ __forceinline__ float gate_value(float z, int act) { return act == 0 ? sigmoid(z) : z * sigmoid(z); }
@@ -46,24 +53,77 @@ struct ScanParams {
   l3ci_recurrent_scan_args a;
   int splits, cols;              // column runs per head, columns per run
   int consumers;                 // warps
-  int vec;                       // q, k, g (and their fp32 companions) allow accesses of four elements
+  int ring;                      // stages
+  int bulk;                      // the tokens' rows can be fetched by bulk tensor copies
+  int wide;                      // state rows allow accesses of four columns
 };
 
-// Four channels from d on, zeros behind the last one (loaded from a place that exists, so that no load hangs on a branch).
-template <typename S>
-__device__ __forceinline__ float4 fetch4(const S* p, int d, int D, int vec) {
-  float f[4];
-  if (vec) {
-    load_vec<S, 4>(p + (d < D ? d : 0), f);
+// Bytes of a stage, part by part: q, k, g as they come, the decays (time mixing), v, two scalars per token.
+template <typename S, typename Q, int KIND, int DP>
+struct ScanStage {
+  static constexpr int kQ = kChunk * DP * (int)sizeof(Q);
+  static constexpr int kK = kQ, kG = kQ;
+  static constexpr int kDecay = KIND == kTimeMix ? kChunk * DP * 4 : 0;
+  static constexpr int kV0 = kQ + kK + kG + kDecay;
+  static constexpr int kScalars = kChunk * 2 * 4;
+  __host__ __device__ static constexpr int bytes(int cols) { return kV0 + kChunk * cols * (int)sizeof(S) + kScalars; }
+  __host__ __device__ static constexpr int loaded(int cols) { return kQ + kK + kG + kChunk * cols * (int)sizeof(S); }
+};
+
+// NR rows of a lane as pairs: rows i * 32 * W + lane * W + e, W = min(NR, 4) neighbours.
+template <typename Q, int NR>
+__device__ __forceinline__ void load_rows(const Q* p, int lane, unsigned long long (&r)[NR / 2]) {
+  constexpr int W = NR < 4 ? NR : 4;
 #pragma unroll
-    for (int e = 0; e < 4; ++e) f[e] = d < D ? f[e] : 0.f;
-  } else {
+  for (int i = 0; i < NR / W; ++i) {
+    const Q* at = p + i * 32 * W + lane * W;
+    if constexpr (sizeof(Q) == 4) {
+      if constexpr (W == 4) {
+        const ulonglong2 x = *reinterpret_cast<const ulonglong2*>(at);
+        r[2 * i] = x.x;
+        r[2 * i + 1] = x.y;
+      } else {
+        r[i] = *reinterpret_cast<const unsigned long long*>(at);
+      }
+    } else {
 #pragma unroll
-    for (int e = 0; e < 4; ++e) f[e] = to_f32(p[d + e < D ? d + e : 0]);
-#pragma unroll
-    for (int e = 0; e < 4; ++e) f[e] = d + e < D ? f[e] : 0.f;
+      for (int e = 0; e < W / 2; ++e) {
+        const uint32_t x = reinterpret_cast<const uint32_t*>(at)[e];
+        r[i * (W / 2) + e] = f2_packf(bf16lo_to_f32(x), bf16hi_to_f32(x));
+      }
+    }
   }
-  return make_float4(f[0], f[1], f[2], f[3]);
+}
+template <int N>
+__device__ __forceinline__ float pairs_dot(const unsigned long long (&a)[N], const unsigned long long (&b)[N]) {
+  unsigned long long s[2] = {0ull, 0ull};
+#pragma unroll
+  for (int j = 0; j < N; ++j) s[j & 1] = f2_fma(a[j], b[j], s[j & 1]);
+  float x, y;
+  f2_unpack(N > 1 ? f2_add(s[0], s[1]) : s[0], x, y);
+  return x + y;
+}
+
+// Sums over the lanes of N values each (a power of two up to 32), halved lane by lane: the lanes of value i are i * 32 / N
+// onwards, and all of them end with its sum.
+template <int N>
+__device__ __forceinline__ float scatter_sum(float (&v)[N], int lane) {
+  int m = 16;
+#pragma unroll
+  for (int n = N / 2; n >= 1; n /= 2, m /= 2) {
+    const bool upper = lane & m;
+#pragma unroll
+    for (int i = 0; i < N / 2; ++i) {
+      if (i >= n) break;
+      const float send = upper ? v[i] : v[i + n], mine = upper ? v[i + n] : v[i];
+      v[i] = mine + __shfl_xor_sync(kFullMask, send, m);
+    }
+  }
+  float r = v[0];
+#pragma unroll
+  for (int k = 16; k >= 1; k /= 2)
+    if (k < 32 / N) r += __shfl_xor_sync(kFullMask, r, k);
+  return r;
 }
 
 // The convolution's carried inputs: row r of the tail becomes the input of token T - (taps - 1) + r.  Channel c of a sequence,
@@ -91,226 +151,352 @@ __device__ __forceinline__ void move_tails(const l3ci_recurrent_scan_args& a, in
 
 // S: storage type of v, gate, out; Q: type of q, k, g.
 template <typename S, typename Q, int KIND, int NR, int C>
-__global__ void __launch_bounds__(kScanThreads) recurrent_scan_kernel(const __grid_constant__ ScanParams p) {
-  constexpr int DP = NR * 8;
-  extern __shared__ __align__(16) float smem[];
+__global__ void __launch_bounds__(32 * (kMaxConsumers[KIND] + 1 + kHelpers[KIND]), 1)
+recurrent_scan_kernel(const __grid_constant__ CUtensorMap qmap, const __grid_constant__ CUtensorMap kmap, const __grid_constant__ CUtensorMap gmap,
+                      const __grid_constant__ CUtensorMap vmap, const __grid_constant__ ScanParams p) {
+  constexpr int DP = 32 * NR;
+  using St = ScanStage<S, Q, KIND, DP>;
+  constexpr int kHelp = kHelpers[KIND];
+  extern __shared__ __align__(128) uint8_t smem_raw[];
+  uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 127) & ~uintptr_t(127));
   const l3ci_recurrent_scan_args& a = p.a;
-  const int cols = p.cols;
-  const int stage_floats = kChunk * (3 * DP + cols + 2);
-  float* stages = smem;
-  uint64_t* bars = reinterpret_cast<uint64_t*>(smem + kRing * stage_floats);
-  const uint32_t full0 = smem_u32(bars), empty0 = full0 + kRing * 8;
+  const int cols = p.cols, stage_bytes = St::bytes(cols), ring = p.ring;
+  uint64_t* bars = reinterpret_cast<uint64_t*>(smem + ring * stage_bytes);
+  const uint32_t full0 = smem_u32(bars), ready0 = full0 + kMaxRing * 8, empty0 = ready0 + kMaxRing * 8;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int split = blockIdx.x % p.splits, h = (blockIdx.x / p.splits) % a.H, b = blockIdx.x / (p.splits * a.H);
   const int D = a.D, V = a.V, T = a.T, R = a.H / a.G, col0 = split * cols;
   if (tid == 0) {
-    for (int i = 0; i < kRing; ++i) {
-      mbar_init(full0 + i * 8, kProducers);
+    for (int i = 0; i < ring; ++i) {
+      mbar_init(full0 + i * 8, 1);
+      mbar_init(ready0 + i * 8, kHelp);
       mbar_init(empty0 + i * 8, p.consumers);
     }
     asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+    asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
   }
   __syncthreads();
   pdl_wait();
   pdl_launch_dependents();
   const bool fresh = a.positions[b] == 0;
   const int chunks = (T + kChunk - 1) / kChunk;
+  const long long row0 = (long long)b * T;
   bool ok = true;
 
-  if (warp >= p.consumers) {
-    // ---- producers ----
-    const int pw = warp - p.consumers;
-    const long long row0 = (long long)b * T;
-    const Q* qp = static_cast<const Q*>(a.q) + (h / R) * a.qk_sh;
-    const Q* kp = static_cast<const Q*>(a.k) + (h / R) * a.qk_sh;
-    const Q* gp = static_cast<const Q*>(a.g) + h * a.g_sh;
-    const S* vp = static_cast<const S*>(a.v) + h * a.v_sh + col0;
-    const int n_cols = min(cols, V - col0);
-    constexpr int kWide = (DP + 127) / 128;      // accesses of four channels per lane and row
-    constexpr int kCols = 4;                     // value columns per lane (a CTA has at most 128)
-    float4 q[kPerProducer][kWide], k[kPerProducer][kWide], g[kPerProducer][kWide];
-    float v[kPerProducer][kCols], beta[kPerProducer];
-    // all loads of this warp's tokens of chunk i (tokens behind the last one: the last one's, never used)
-    auto fetch = [&](int i) {
-#pragma unroll
-      for (int x = 0; x < kPerProducer; ++x) {
-        const long long row = row0 + min(i * kChunk + pw * kPerProducer + x, T - 1);
-#pragma unroll
-        for (int j = 0; j < kWide; ++j) {
-          const int d = j * 128 + lane * 4;
-          q[x][j] = fetch4<Q>(qp + row * a.qk_st, d, D, p.vec);
-          k[x][j] = fetch4<Q>(kp + row * a.qk_st, d, D, p.vec);
-          g[x][j] = fetch4<Q>(gp + row * a.g_st, d, D, p.vec);
+  if (warp == p.consumers) {
+    // ---- producer ----
+    const uint64_t policy = l2_evict_first_policy();
+    for (int i = 0, s = 0, phase = 1; i < chunks; ++i, s = s + 1 == ring ? 0 : s + 1, phase ^= s == 0) {
+      if (i >= ring && !mbar_wait_bounded(empty0 + s * 8, phase)) { ok = false; break; }
+      uint8_t* st = smem + s * stage_bytes;
+      if (p.bulk) {
+        if (lane == 0) {
+          const uint32_t bar = full0 + s * 8, dst = smem_u32(st);
+          mbar_expect_tx(bar, St::loaded(cols));
+          tma_load_4d(dst, &qmap, bar, 0, i * kChunk, h / R, b, policy);
+          tma_load_4d(dst + St::kQ, &kmap, bar, 0, i * kChunk, h / R, b, policy);
+          tma_load_4d(dst + St::kQ + St::kK, &gmap, bar, 0, i * kChunk, h, b, policy);
+          tma_load_4d(dst + St::kV0, &vmap, bar, col0, i * kChunk, h, b, policy);
         }
-#pragma unroll
-        for (int c = 0; c < kCols; ++c) v[x][c] = to_f32(vp[row * a.v_st + min(c * 32 + lane, n_cols - 1)]);
-        beta[x] = KIND == kDelta ? a.beta[row * a.H + h] : 0.f;
-      }
-    };
-    float4 bonus[kWide], gb[kWide];
-    if (KIND == kTimeMix) {
-#pragma unroll
-      for (int j = 0; j < kWide; ++j) {
-        bonus[j] = fetch4<float>(a.bonus + h * D, j * 128 + lane * 4, D, p.vec);
-        gb[j] = fetch4<float>(a.g_bias + h * D, j * 128 + lane * 4, D, p.vec);
-      }
-    }
-    fetch(0);
-    for (int i = 0; i < chunks; ++i) {
-      const int s = i % kRing;
-      if (i >= kRing && !mbar_wait_bounded(empty0 + s * 8, ((i / kRing) - 1) & 1)) { ok = false; break; }
-      float* st = stages + s * stage_floats;
-      float* vs = st + kChunk * 3 * DP;
-      float* sc = vs + kChunk * cols;
-      float scalar[kPerProducer];
-#pragma unroll
-      for (int x = 0; x < kPerProducer; ++x) {
-        const int at = pw * kPerProducer + x;
-        scalar[x] = 0.f;
-#pragma unroll
-        for (int j = 0; j < kWide; ++j) {
-          const int d = j * 128 + lane * 4;
-          const float4 qq = q[x][j], kk = k[x][j];
-          float4 gg = g[x][j];
-          if (KIND == kTimeMix) {
-            gg.x = expf(-expf(gg.x + gb[j].x));
-            gg.y = expf(-expf(gg.y + gb[j].y));
-            gg.z = expf(-expf(gg.z + gb[j].z));
-            gg.w = expf(-expf(gg.w + gb[j].w));
-            scalar[x] += qq.x * kk.x * bonus[j].x + qq.y * kk.y * bonus[j].y + qq.z * kk.z * bonus[j].z + qq.w * kk.w * bonus[j].w;
-          } else {
-            scalar[x] += qq.x * kk.x + qq.y * kk.y + qq.z * kk.z + qq.w * kk.w;
+      } else {
+        const int n = min(kChunk, T - i * kChunk);
+        Q *qs = reinterpret_cast<Q*>(st), *ks = qs + kChunk * DP, *gs = ks + kChunk * DP;
+        S* vs = reinterpret_cast<S*>(st + St::kV0);
+        for (int x = 0; x < n; ++x) {
+          const long long row = row0 + i * kChunk + x;
+          for (int d = lane; d < DP; d += 32) {
+            const bool in = d < D;
+            qs[x * DP + d] = in ? static_cast<const Q*>(a.q)[row * a.qk_st + (h / R) * a.qk_sh + d] : from_f32<Q>(0.f);
+            ks[x * DP + d] = in ? static_cast<const Q*>(a.k)[row * a.qk_st + (h / R) * a.qk_sh + d] : from_f32<Q>(0.f);
+            gs[x * DP + d] = in ? static_cast<const Q*>(a.g)[row * a.g_st + h * a.g_sh + d] : from_f32<Q>(0.f);
           }
-          if (d < DP) {
-            float* row = st + at * 3 * DP + d;
-            *reinterpret_cast<float4*>(row) = qq;
-            *reinterpret_cast<float4*>(row + DP) = kk;
-            *reinterpret_cast<float4*>(row + 2 * DP) = gg;
-          }
+          for (int c = lane; c < cols; c += 32)
+            vs[x * cols + c] = col0 + c < V ? static_cast<const S*>(a.v)[row * a.v_st + h * a.v_sh + col0 + c] : from_f32<S>(0.f);
         }
-#pragma unroll
-        for (int c = 0; c < kCols; ++c)
-          if (c * 32 + lane < cols) vs[at * cols + c * 32 + lane] = c * 32 + lane < n_cols ? v[x][c] : 0.f;
-      }
-#pragma unroll
-      for (int x = 0; x < kPerProducer; ++x) scalar[x] = group_sum<kWarp>(scalar[x]);
-      if (lane == 0) {
-#pragma unroll
-        for (int x = 0; x < kPerProducer; ++x) {
-          sc[(pw * kPerProducer + x) * 2] = scalar[x];
-          sc[(pw * kPerProducer + x) * 2 + 1] = beta[x];
-        }
+        __syncwarp();
+        if (lane == 0) mbar_arrive(full0 + s * 8);
       }
       __syncwarp();
-      if (lane == 0) mbar_arrive(full0 + s * 8);
-      if (i + 1 < chunks) fetch(i + 1);
     }
-    if (a.tail && split == 0) move_tails<S>(a, b, h, pw * 32 + lane, 32 * kProducers, fresh);
+    if (a.tail && split == 0) move_tails<S>(a, b, h, lane, 32, fresh);
     if (!ok && lane == 0 && a.status) atomicExch(a.status, (int)L3CI_ERR_DEVICE_WAIT);
     return;
   }
 
-  // ---- consumers: lane l of a group of 8 holds rows 32 i + 4 l + e of the group's C columns ----
-  const int l = lane & 7, c_loc = (warp * 4 + (lane >> 3)) * C, c0 = col0 + c_loc;
-  const bool live = c_loc < cols && c0 < V;    // (V and cols are multiples of C)
+  if (warp > p.consumers) {
+    // ---- helpers ----
+    const int hw = warp - p.consumers - 1;
+    unsigned long long k_before[NR / 2], gb[NR / 2];
+#pragma unroll
+    for (int j = 0; j < NR / 2; ++j) k_before[j] = gb[j] = 0ull;
+    if (KIND == kTimeMix) {
+      constexpr int W = NR < 4 ? NR : 4;
+#pragma unroll
+      for (int j = 0; j < NR / 2; ++j) {
+        const int d = (2 * j / W) * 32 * W + lane * W + 2 * j % W;
+        gb[j] = f2_packf(d < D ? a.g_bias[h * D + d] : 0.f, d + 1 < D ? a.g_bias[h * D + d + 1] : 0.f);
+      }
+    }
+    auto step_size = [&](int i) {      // of token `lane` of chunk i
+      return KIND == kDelta && lane < kChunk ? a.beta[(row0 + min(i * kChunk + lane, T - 1)) * a.H + h] : 0.f;
+    };
+    float beta = step_size(0);
+    for (int i = 0, s = 0, phase = 0; i < chunks; ++i, s = s + 1 == ring ? 0 : s + 1, phase ^= s == 0) {
+      if (!mbar_wait_bounded(full0 + s * 8, phase)) { ok = false; break; }
+      uint8_t* st = smem + s * stage_bytes;
+      if (KIND == kDelta) {
+        const Q *ks = reinterpret_cast<const Q*>(st + St::kQ), *gs = reinterpret_cast<const Q*>(st + St::kQ + St::kK);
+        float part[kChunk];
+#pragma unroll
+        for (int x = 0; x < kChunk; ++x) {
+          unsigned long long k[NR / 2], g[NR / 2];
+          load_rows<Q, NR>(ks + x * DP, lane, k);
+          load_rows<Q, NR>(gs + x * DP, lane, g);
+#pragma unroll
+          for (int j = 0; j < NR / 2; ++j) {
+            g[j] = f2_mul(g[j], k[j]);
+          }
+          part[x] = pairs_dot(g, k_before);
+#pragma unroll
+          for (int j = 0; j < NR / 2; ++j) k_before[j] = k[j];
+        }
+        const float sum = scatter_sum<kChunk>(part, lane);       // lanes 2 x, 2 x + 1: token x
+        float* sc = reinterpret_cast<float*>(st + stage_bytes - St::kScalars);
+        if (lane % 2 == 0) sc[lane + 1] = sum;
+        if (lane < kChunk) sc[2 * lane] = beta;
+        beta = step_size(min(i + 1, chunks - 1));
+      } else {
+        const Q* gs = reinterpret_cast<const Q*>(st + St::kQ + St::kK);
+        float* ds = reinterpret_cast<float*>(st + St::kQ + St::kK + St::kG);
+        constexpr int W = NR < 4 ? NR : 4;
+#pragma unroll
+        for (int x0 = 0; x0 < kChunk / kHelp; ++x0) {
+          const int x = x0 * kHelp + hw;
+          unsigned long long g[NR / 2];
+          load_rows<Q, NR>(gs + x * DP, lane, g);
+#pragma unroll
+          for (int j = 0; j < NR / 2; ++j) {
+            float u, v;
+            f2_unpack(f2_add(g[j], gb[j]), u, v);
+            *reinterpret_cast<unsigned long long*>(ds + x * DP + (2 * j / W) * 32 * W + lane * W + 2 * j % W) = f2_packf(expf(-expf(u)), expf(-expf(v)));
+          }
+        }
+      }
+      __syncwarp();
+      if (lane == 0) mbar_arrive(ready0 + s * 8);
+    }
+    if (!ok && lane == 0 && a.status) atomicExch(a.status, (int)L3CI_ERR_DEVICE_WAIT);
+    return;
+  }
+
+  // ---- consumers ----
+  constexpr int W = NR < 4 ? NR : 4;
+  constexpr int kBlock = 32 / C;                 // tokens whose outputs are summed together
+  constexpr int kShift = KIND == kDelta ? 1 : 0; // the delta rule writes a token's output while it takes the next one
+  const int c_loc = warp * C, c0 = col0 + c_loc;
   float* state = a.state + b * a.state_sb + (long long)h * D * V + c0;
-  unsigned long long S2[C][NR / 2];            // rows in pairs
+  const bool wide = p.wide && c0 + C <= V;
+  unsigned long long A[C][NR / 2];
+  auto row_of = [&](int j) { return (2 * j / W) * 32 * W + lane * W + 2 * j % W; };   // first row of pair j
 #pragma unroll
-  for (int i = 0; i < NR / 4; ++i) {
-    float f[4][C];
+  for (int j = 0; j < NR / 2; ++j) {
+    float f[2][C];
 #pragma unroll
-    for (int e = 0; e < 4; ++e) {
+    for (int e = 0; e < 2; ++e) {
+      const int row = row_of(j) + e;
 #pragma unroll
       for (int c = 0; c < C; ++c) f[e][c] = 0.f;
-      const int row = 32 * i + 4 * l + e;
-      if (live && !fresh && row < D) load_vec<float, C>(state + (long long)row * V, f[e]);
+      if (fresh || row >= D) continue;
+      const float* at = state + (long long)row * V;
+      if (wide) {
+#pragma unroll
+        for (int c = 0; c < C; c += 4) {
+          const float4 x = *reinterpret_cast<const float4*>(at + c);
+          f[e][c] = x.x; f[e][c + 1] = x.y; f[e][c + 2] = x.z; f[e][c + 3] = x.w;
+        }
+      } else {
+#pragma unroll
+        for (int c = 0; c < C; ++c)
+          if (c0 + c < V) f[e][c] = at[c];
+      }
     }
 #pragma unroll
-    for (int c = 0; c < C; ++c) {
-      S2[c][2 * i] = f2_packf(f[0][c], f[1][c]);
-      S2[c][2 * i + 1] = f2_packf(f[2][c], f[3][c]);
+    for (int c = 0; c < C; ++c) A[c][j] = f2_packf(f[0][c], f[1][c]);
+  }
+  // carried from the token before (delta rule): k, q, its value, step size, scalar and sum over the state of this lane's
+  // column, and the u of the token before that
+  unsigned long long kp[NR / 2], qp[NR / 2];
+  float v_p = 0.f, beta_p = 0.f, cross_p = 0.f, seen_p = 0.f, u_p = 0.f;
+#pragma unroll
+  for (int j = 0; j < NR / 2; ++j) kp[j] = qp[j] = 0ull;
+  unsigned long long bonus[NR / 2];
+  if (KIND == kTimeMix) {
+#pragma unroll
+    for (int j = 0; j < NR / 2; ++j) {
+      const int d = row_of(j);
+      bonus[j] = f2_packf(d < D ? a.bonus[h * D + d] : 0.f, d + 1 < D ? a.bonus[h * D + d + 1] : 0.f);
     }
   }
-  S* out = static_cast<S*>(a.out) + (long long)b * T * a.out_st + h * a.out_sh + c0;
-  float o[C];
-  for (int i = 0; i < chunks; ++i) {
-    const int s = i % kRing, n = min(kChunk, T - i * kChunk);
-    if (!mbar_wait_bounded(full0 + s * 8, (i / kRing) & 1)) { ok = false; break; }
-    const float* st = stages + s * stage_floats + 4 * l;
-    const float* vs = stages + s * stage_floats + kChunk * 3 * DP + (live ? c_loc : 0);
-    const float* sc = stages + s * stage_floats + kChunk * (3 * DP + cols);
-#pragma unroll 2
-    for (int x = 0; x < n; ++x, st += 3 * DP, vs += cols, sc += 2) {
-      unsigned long long q2[NR / 2], k2[NR / 2], g2[NR / 2];
+  S* out = static_cast<S*>(a.out) + row0 * a.out_st + h * a.out_sh + c0;
+  // the warp's patch: this lane's shares of the outputs, C floats per token
+  float* patch = reinterpret_cast<float*>(smem + ring * stage_bytes + 3 * kMaxRing * 8 + warp * kPatchBytes);
+  // (stored behind the block's last token: between the tokens the stores would hold up the loads of the next one)
+  auto share = [&](int x, const float* part) {
 #pragma unroll
-      for (int j = 0; j < NR / 4; ++j) {
-        const ulonglong2 qq = *reinterpret_cast<const ulonglong2*>(st + 32 * j);
-        const ulonglong2 kk = *reinterpret_cast<const ulonglong2*>(st + DP + 32 * j);
-        const ulonglong2 gg = *reinterpret_cast<const ulonglong2*>(st + 2 * DP + 32 * j);
-        q2[2 * j] = qq.x; q2[2 * j + 1] = qq.y;
-        k2[2 * j] = kk.x; k2[2 * j + 1] = kk.y;
-        g2[2 * j] = gg.x; g2[2 * j + 1] = gg.y;
+    for (int c = 0; c < C; c += 4)
+      *reinterpret_cast<float4*>(patch + x * kPatchToken<C> + c / 4 * 128 + lane * 4) = make_float4(part[c], part[c + 1], part[c + 2], part[c + 3]);
+  };
+  // the outputs of the block's n tokens from t0 on: C lanes per token sum the shares of 32 / C lanes each, all columns, and
+  // then halve the columns among themselves
+  auto write = [&](int t0, int n) {
+    __syncwarp();
+    const int x = lane / C, part = lane % C;
+    float sums[C];
+#pragma unroll
+    for (int c = 0; c < C; ++c) sums[c] = 0.f;
+#pragma unroll
+    for (int i = 0; i < 32 / C; ++i)
+#pragma unroll
+      for (int c = 0; c < C; c += 4) {
+        const float4 y = *reinterpret_cast<const float4*>(patch + x * kPatchToken<C> + c / 4 * 128 + (i * C + part) * 4);
+        sums[c] += y.x; sums[c + 1] += y.y; sums[c + 2] += y.z; sums[c + 3] += y.w;
       }
-      const float scalar = sc[0], beta = sc[1];
-      float v[C], dk[C], dq[C];
+#pragma unroll
+    for (int m = C / 2; m >= 1; m /= 2) {
+      const bool upper = part & m;
+#pragma unroll
+      for (int c = 0; c < m; ++c) {
+        const float send = upper ? sums[c] : sums[c + m], mine = upper ? sums[c + m] : sums[c];
+        sums[c] = mine + __shfl_xor_sync(kFullMask, send, m);
+      }
+    }
+    const int t = t0 + x - kShift;
+    if (x < n && t >= 0 && c0 + part < V) out[t * a.out_st + part] = from_f32<S>(sums[0]);
+    __syncwarp();
+  };
+  // u of the token before, now that its sum over the state is there: this lane's column, then every column, twice
+  auto finish = [&](unsigned long long (&ub)[C]) {
+    u_p = beta_p * (v_p - fmaf(cross_p, u_p, seen_p));
+#pragma unroll
+    for (int c = 0; c < C; ++c) {
+      const float u = __shfl_sync(kFullMask, u_p, c * (32 / C));
+      ub[c] = f2_packf(u, u);
+    }
+  };
+  // token x of the stage; part: this lane's shares of the outputs
+  auto token = [&](const uint8_t* st, int x, float* part) {
+    unsigned long long q[NR / 2], k[NR / 2], g[NR / 2];
+    load_rows<Q, NR>(reinterpret_cast<const Q*>(st) + x * DP, lane, q);
+    load_rows<Q, NR>(reinterpret_cast<const Q*>(st + St::kQ) + x * DP, lane, k);
+    load_rows<float, NR>(reinterpret_cast<const float*>(st + St::kQ + St::kK + (KIND == kTimeMix ? St::kG : 0)) + x * DP, lane, g);
+    const S* vs = reinterpret_cast<const S*>(st + St::kV0) + x * cols + c_loc;
+    if constexpr (KIND == kDelta) {
+      const float* sc = reinterpret_cast<const float*>(st + stage_bytes - St::kScalars) + 2 * x;
+      unsigned long long ub[C], gk[NR / 2];
+      finish(ub);
+#pragma unroll
+      for (int j = 0; j < NR / 2; ++j) gk[j] = f2_mul(g[j], k[j]);
+      float sums[C];
+#pragma unroll
+      for (int c = 0; c < C; ++c) sums[c] = pairs_dot(gk, A[c]);
+      seen_p = scatter_sum<C>(sums, lane);
 #pragma unroll
       for (int c = 0; c < C; ++c) {
-        v[c] = vs[c];
-        // two chains each
-        unsigned long long aq[2] = {0ull, 0ull}, ak[2] = {0ull, 0ull};
+#pragma unroll
+        for (int j = 0; j < NR / 2; ++j) A[c][j] = f2_fma(kp[j], ub[c], A[c][j]);       // S_{t-1}
+        part[c] = pairs_dot(qp, A[c]);
+#pragma unroll
+        for (int j = 0; j < NR / 2; ++j) A[c][j] = f2_mul(A[c][j], g[j]);               // S'_t
+      }
+      v_p = to_f32(vs[lane / (32 / C)]);
+      beta_p = sc[0];
+      cross_p = sc[1];
+#pragma unroll
+      for (int j = 0; j < NR / 2; ++j) {
+        kp[j] = k[j];
+        qp[j] = q[j];
+      }
+    } else {
+      unsigned long long qb[NR / 2];
+#pragma unroll
+      for (int j = 0; j < NR / 2; ++j) qb[j] = f2_mul(f2_mul(q[j], bonus[j]), k[j]);
+      float v[C];
+      load_vec<S, 4>(vs, reinterpret_cast<float(&)[4]>(v[0]));
+      if constexpr (C == 8) load_vec<S, 4>(vs + 4, reinterpret_cast<float(&)[4]>(v[4]));
+#pragma unroll
+      for (int c = 0; c < C; ++c) {
+        const unsigned long long v2 = f2_packf(v[c], v[c]);
+        unsigned long long sum = 0ull;
 #pragma unroll
         for (int j = 0; j < NR / 2; ++j) {
-          if (KIND == kDelta) {
-            S2[c][j] = f2_mul(S2[c][j], g2[j]);
-            ak[j & 1] = f2_fma(S2[c][j], k2[j], ak[j & 1]);
-          }
-          aq[j & 1] = f2_fma(S2[c][j], q2[j], aq[j & 1]);
+          sum = f2_fma(q[j], A[c][j], f2_fma(qb[j], v2, sum));
+          A[c][j] = f2_fma(k[j], v2, f2_mul(A[c][j], g[j]));
         }
-        float x0, x1;
-        f2_unpack(f2_add(aq[0], aq[1]), x0, x1);
-        dq[c] = x0 + x1;
-        if (KIND == kDelta) {
-          f2_unpack(f2_add(ak[0], ak[1]), x0, x1);
-          dk[c] = x0 + x1;
+        float y, z;
+        f2_unpack(sum, y, z);
+        part[c] = y + z;
+      }
+    }
+  };
+  for (int i = 0, s = 0, phase = 0; i < chunks; ++i, s = s + 1 == ring ? 0 : s + 1, phase ^= s == 0) {
+    const int n = min(kChunk, T - i * kChunk);
+    if (!mbar_wait_bounded(ready0 + s * 8, phase) || !mbar_wait_bounded(full0 + s * 8, phase)) { ok = false; break; }
+    const uint8_t* st = smem + s * stage_bytes;
+    for (int x0 = 0; x0 < n; x0 += kBlock) {
+      if (n - x0 >= kBlock) {
+        float part[kBlock * C];
+#pragma unroll
+        for (int x = 0; x < kBlock; ++x) token(st, x0 + x, part + x * C);
+#pragma unroll
+        for (int x = 0; x < kBlock; ++x) share(x, part + x * C);
+        write(i * kChunk + x0, kBlock);
+      } else {
+        for (int x = 0; x < n - x0; ++x) {
+          float part[C];
+          token(st, x0 + x, part);
+          share(x, part);
         }
+        write(i * kChunk + x0, n - x0);
       }
-#pragma unroll
-      for (int c = 0; c < C; ++c) {
-        if (KIND == kDelta) dk[c] = group_sum<8>(dk[c]);
-        dq[c] = group_sum<8>(dq[c]);
-      }
-#pragma unroll
-      for (int c = 0; c < C; ++c) {
-        const float u = KIND == kDelta ? beta * (v[c] - dk[c]) : v[c];
-        o[c] = fmaf(scalar, u, dq[c]);
-        const unsigned long long u2 = f2_packf(u, u);
-#pragma unroll
-        for (int j = 0; j < NR / 2; ++j) S2[c][j] = f2_fma(k2[j], u2, KIND == kDelta ? S2[c][j] : f2_mul(S2[c][j], g2[j]));
-      }
-      if (l == 0 && live) {
-#pragma unroll
-        for (int c = 0; c < C; ++c) out[c] = from_f32<S>(o[c]);
-      }
-      out += a.out_st;
     }
     __syncwarp();
     if (lane == 0) mbar_arrive(empty0 + s * 8);
   }
   if (!ok) {
     if (lane == 0 && a.status) atomicExch(a.status, (int)L3CI_ERR_DEVICE_WAIT);
-  } else {
+    return;
+  }
+  if (KIND == kDelta) {
+    // the last token's write and output
+    unsigned long long ub[C];
+    finish(ub);
+    float part[C];
 #pragma unroll
-    for (int i = 0; i < NR / 4; ++i) {
-      float f[4][C];
+    for (int c = 0; c < C; ++c) {
 #pragma unroll
-      for (int c = 0; c < C; ++c) {
-        f2_unpack(S2[c][2 * i], f[0][c], f[1][c]);
-        f2_unpack(S2[c][2 * i + 1], f[2][c], f[3][c]);
-      }
+      for (int j = 0; j < NR / 2; ++j) A[c][j] = f2_fma(kp[j], ub[c], A[c][j]);
+      part[c] = pairs_dot(qp, A[c]);
+    }
+    share(0, part);
+    write(T, 1);
+  }
 #pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        const int row = 32 * i + 4 * l + e;
-        if (live && row < D) store_vec<float, C>(state + (long long)row * V, f[e]);
+  for (int j = 0; j < NR / 2; ++j) {
+    float f[2][C];
+#pragma unroll
+    for (int c = 0; c < C; ++c) f2_unpack(A[c][j], f[0][c], f[1][c]);
+#pragma unroll
+    for (int e = 0; e < 2; ++e) {
+      const int row = row_of(j) + e;
+      if (row >= D) continue;
+      float* at = state + (long long)row * V;
+      if (wide) {
+#pragma unroll
+        for (int c = 0; c < C; c += 4) *reinterpret_cast<float4*>(at + c) = make_float4(f[e][c], f[e][c + 1], f[e][c + 2], f[e][c + 3]);
+      } else {
+#pragma unroll
+        for (int c = 0; c < C; ++c)
+          if (c0 + c < V) at[c] = f[e][c];
       }
     }
   }
@@ -424,7 +610,40 @@ __global__ void __launch_bounds__(kStepThreads, RP <= 4 ? 5 : RP <= 8 ? 3 : 2) r
   if (a.tail) move_tails<S>(a, b, h, tid, kStepThreads, fresh);
 }
 
-// out[row, h, :] <- out / rms(out) * norm * act(gate), in place: a warp per (row, head)
+// out[row, h, :] <- out / rms(out) * norm * act(gate), in place: LANES lanes per (row, head), a vector per lane
+template <typename S, int VEC, int LANES>
+__global__ void __launch_bounds__(256)
+head_norm_gate_vec_kernel(S* __restrict__ out, long long out_st, long long out_sh, const S* __restrict__ gate, long long gate_st,
+                          long long gate_sh, const float* __restrict__ norm, long long norm_sh, int H, int V, long long units, int act, float eps) {
+  pdl_wait();
+  pdl_launch_dependents();
+  const long long id = (long long)blockIdx.x * (256 / LANES) + threadIdx.x / LANES;
+  const int c = (threadIdx.x % LANES) * VEC;
+  const bool mine = id < units && c < V;
+  const long long row = units <= 0xffffffffLL ? (unsigned)id / (unsigned)H : id / H;
+  const int h = (int)(id - row * H);
+  float x[VEC], z[VEC], w[VEC];
+#pragma unroll
+  for (int k = 0; k < VEC; ++k) x[k] = 0.f;
+  if (mine) {
+    load_vec<S, VEC>(out + row * out_st + h * out_sh + c, x);
+    load_vec<S, VEC>(gate + row * gate_st + h * gate_sh + c, z);
+    load_vec<float, VEC>(norm + h * norm_sh + c, w);
+  }
+  float ss = 0.f;
+#pragma unroll
+  for (int k = 0; k < VEC; ++k) ss = fmaf(x[k], x[k], ss);
+  const float inv = 1.f / sqrtf(group_sum<LANES>(ss) / (float)V + eps);
+  if (!mine) return;
+#pragma unroll
+  for (int k = 0; k < VEC; ++k) {
+    const float s = sizeof(S) == 4 ? sigmoid(z[k]) : __fdividef(1.f, 1.f + __expf(-z[k]));
+    x[k] = x[k] * inv * w[k] * (act == 0 ? s : z[k] * s);
+  }
+  store_vec<S, VEC>(out + row * out_st + h * out_sh + c, x);
+}
+
+// The same for any size: a warp per (row, head)
 template <typename S, int VEC>
 __global__ void __launch_bounds__(256)
 head_norm_gate_kernel(S* __restrict__ out, long long out_st, long long out_sh, const S* __restrict__ gate, long long gate_st,
@@ -627,17 +846,31 @@ __global__ void __launch_bounds__(256) delta_inputs_kernel(const l3ci_delta_inpu
 constexpr int kMaxD = 256;         // key channels of a head
 
 template <typename S, typename Q, int KIND, int NR, int C>
-int launch_scan(const ScanParams& p, cudaStream_t stream) {
-  const size_t smem = (size_t)kRing * kChunk * (3 * NR * 8 + p.cols + 2) * 4 + 2 * kRing * 8;
+int launch_scan(ScanParams p, cudaStream_t stream) {
+  constexpr int DP = 32 * NR;
+  using St = ScanStage<S, Q, KIND, DP>;
+  const l3ci_recurrent_scan_args& a = p.a;
+  const size_t fixed = 128 + 3 * kMaxRing * 8 + (size_t)p.consumers * kPatchBytes;
+  p.ring = (int)((max_smem_optin() - fixed) / St::bytes(p.cols));
+  if (p.ring > kMaxRing) p.ring = kMaxRing;
+  if (p.ring < 1) return fail(L3CI_ERR_UNSUPPORTED, "recurrent_scan: D=%d V=%d", a.D, a.V);
+  const size_t smem = fixed + (size_t)p.ring * St::bytes(p.cols);
   static bool configured[64] = {false};
   int dev = 0;
   L3CI_CUDA_TRY(cudaGetDevice(&dev));
-  if (smem > (48 << 10) && (dev < 0 || dev >= 64 || !configured[dev])) {
+  if (dev < 0 || dev >= 64 || !configured[dev]) {
     L3CI_CUDA_TRY(cudaFuncSetAttribute(recurrent_scan_kernel<S, Q, KIND, NR, C>, cudaFuncAttributeMaxDynamicSharedMemorySize, max_smem_optin()));
     if (dev >= 0 && dev < 64) configured[dev] = true;
   }
-  L3CI_LAUNCH("recurrent_scan_kernel", recurrent_scan_kernel<S, Q, KIND, NR, C>, dim3((unsigned)((long long)p.a.B * p.a.H * p.splits)),
-              dim3(32 * (p.consumers + kProducers)), smem, stream, p);
+  CUtensorMap q = {}, k = {}, g = {}, v = {};
+  if (p.bulk) {
+    if (int st = make_box_map(&q, a.q, sizeof(Q), a.D, a.T, a.G, a.B, a.qk_st, a.qk_sh, a.T * a.qk_st, DP, kChunk)) return st;
+    if (int st = make_box_map(&k, a.k, sizeof(Q), a.D, a.T, a.G, a.B, a.qk_st, a.qk_sh, a.T * a.qk_st, DP, kChunk)) return st;
+    if (int st = make_box_map(&g, a.g, sizeof(Q), a.D, a.T, a.H, a.B, a.g_st, a.g_sh, a.T * a.g_st, DP, kChunk)) return st;
+    if (int st = make_box_map(&v, a.v, sizeof(S), a.V, a.T, a.H, a.B, a.v_st, a.v_sh, a.T * a.v_st, p.cols, kChunk)) return st;
+  }
+  L3CI_LAUNCH("recurrent_scan_kernel", recurrent_scan_kernel<S, Q, KIND, NR, C>, dim3((unsigned)((long long)a.B * a.H * p.splits)),
+              dim3(32 * (p.consumers + 1 + kHelpers[KIND])), smem, stream, q, k, g, v, p);
   return L3CI_OK;
 }
 
@@ -669,52 +902,49 @@ int scan_typed(const l3ci_recurrent_scan_args* a, cudaStream_t stream) {
   p.a = *a;
   const long long heads = (long long)a->B * a->H;
   const int sms = sm_count() > 0 ? sm_count() : 148;
-  // columns per thread: as many as leave enough CTAs for the device
-  const int widest = a->V % 4 == 0 && a->state_sb % 4 == 0 && (reinterpret_cast<uintptr_t>(a->state) & 15) == 0   ? 4
-                     : a->V % 2 == 0 && a->state_sb % 2 == 0 && (reinterpret_cast<uintptr_t>(a->state) & 7) == 0 ? 2
-                                                                                                                 : 1;
-  int C = 1;
-  const struct { int C, W; } shapes[] = {{4, 8}, {2, 8}, {2, 4}, {1, 4}, {1, 2}};
-  for (const auto& s : shapes) {
-    if (s.C > widest && s.C > 1) continue;
+  p.wide = a->V % 4 == 0 && a->state_sb % 4 == 0 && aligned16(a->state);
+  // rows the copy engine can address: whole 16-byte vectors
+  auto rows16 = [](const void* x, size_t size, int64_t st, int64_t sh) { return aligned16(x) && st > 0 && sh > 0 && (st * size) % 16 == 0 && (sh * size) % 16 == 0; };
+  p.bulk = rows16(a->q, sizeof(Q), a->qk_st, a->qk_sh) && rows16(a->k, sizeof(Q), a->qk_st, a->qk_sh) && rows16(a->g, sizeof(Q), a->g_st, a->g_sh) &&
+           rows16(a->v, sizeof(S), a->v_st, a->v_sh);
+  // columns per warp and warps per CTA: as many as leave enough CTAs for the device
+  // (the delta rule wants the registers, time mixing the warps)
+  const struct { int C, W; } by_kind[2][4] = {{{8, 8}, {8, 4}, {4, 4}, {4, 2}}, {{4, 16}, {4, 8}, {4, 4}, {4, 2}}};
+  int C = 4;
+  for (const auto& s : by_kind[KIND]) {
     C = s.C;
     p.consumers = s.W;
-    p.splits = (a->V + 4 * C * s.W - 1) / (4 * C * s.W);
-    if (heads * p.splits * 5 >= 4LL * sms) break;
+    p.cols = C * s.W;
+    p.splits = (a->V + p.cols - 1) / p.cols;
+    if (p.cols < 2 * a->V && heads * p.splits * 5 >= 4LL * sms) break;
   }
-  const int need = (a->V + 4 * C - 1) / (4 * C);
-  if (p.consumers > need) p.consumers = need;
-  p.cols = 4 * C * p.consumers;
-  if (p.splits * (long long)p.cols < a->V) p.splits = (a->V + p.cols - 1) / p.cols;
   if (heads * p.splits > 0x7fffffffLL) return fail(L3CI_ERR_INVALID, "recurrent_scan: too many sequences");
   auto on = [](const void* x, int bytes) { return (reinterpret_cast<uintptr_t>(x) & (bytes - 1)) == 0; };
-  const int q4 = 4 * (int)sizeof(Q);
-  p.vec = a->D % 4 == 0 && (a->qk_st | a->qk_sh | a->g_st | a->g_sh) % 4 == 0 && on(a->q, q4) && on(a->k, q4) && on(a->g, q4) &&
-          on(a->bonus, 16) && on(a->g_bias, 16);
-  auto rows = [&](auto c) -> int {
-    constexpr int CC = decltype(c)::value;
-    if (a->D <= 32) return launch_scan<S, Q, KIND, 4, CC>(p, stream);
-    if (a->D <= 64) return launch_scan<S, Q, KIND, 8, CC>(p, stream);
-    if (a->D <= 128) return launch_scan<S, Q, KIND, 16, CC>(p, stream);
-    return launch_scan<S, Q, KIND, 32, CC>(p, stream);
-  };
   int st;
-  if (C == 4) st = rows(std::integral_constant<int, 4>{});
-  else if (C == 2) st = rows(std::integral_constant<int, 2>{});
-  else st = rows(std::integral_constant<int, 1>{});
+  auto by_rows = [&](auto c) -> int {
+    constexpr int CC = decltype(c)::value;
+    return a->D <= 64 ? launch_scan<S, Q, KIND, 2, CC>(p, stream) : a->D <= 128 ? launch_scan<S, Q, KIND, 4, CC>(p, stream)
+                                                                              : launch_scan<S, Q, KIND, 8, CC>(p, stream);
+  };
+  if constexpr (KIND == kDelta) st = C == 8 ? by_rows(std::integral_constant<int, 8>{}) : by_rows(std::integral_constant<int, 4>{});
+  else st = by_rows(std::integral_constant<int, 4>{});
   if (st) return st;
   // norm and gate of the rows the scan has written
   const long long units = heads * a->T;
   if ((units + 7) / 8 > 0x7fffffffLL) return fail(L3CI_ERR_INVALID, "recurrent_scan: too many rows");
-  const bool v4 = (a->V | a->out_st | a->out_sh | a->gate_st | a->gate_sh | a->norm_sh) % 4 == 0 && on(a->out, 4 * sizeof(S)) &&
-                  on(a->gate, 4 * sizeof(S)) && on(a->norm, 16);
-  auto go = [&](auto kernel) -> int {
-    L3CI_LAUNCH("head_norm_gate_kernel", kernel, dim3((unsigned)((units + 7) / 8)), dim3(256), 0, stream, static_cast<S*>(a->out),
+  auto go = [&](auto kernel, int per_cta) -> int {
+    L3CI_LAUNCH("head_norm_gate_kernel", kernel, dim3((unsigned)((units + per_cta - 1) / per_cta)), dim3(256), 0, stream, static_cast<S*>(a->out),
                 (long long)a->out_st, (long long)a->out_sh, static_cast<const S*>(a->gate), (long long)a->gate_st, (long long)a->gate_sh,
                 a->norm, (long long)a->norm_sh, a->H, a->V, units, a->act, a->eps);
     return L3CI_OK;
   };
-  return v4 ? go(head_norm_gate_kernel<S, 4>) : go(head_norm_gate_kernel<S, 1>);
+  constexpr int kVec = 16 / sizeof(S);
+  const bool vec = (a->V | a->out_st | a->out_sh | a->gate_st | a->gate_sh | a->norm_sh) % kVec == 0 && aligned16(a->out) && aligned16(a->gate) &&
+                   aligned16(a->norm);
+  if (vec && a->V <= 8 * kVec) return go(head_norm_gate_vec_kernel<S, kVec, 8>, 32);
+  if (vec && a->V <= 16 * kVec) return go(head_norm_gate_vec_kernel<S, kVec, 16>, 16);
+  if (vec && a->V <= 32 * kVec) return go(head_norm_gate_vec_kernel<S, kVec, 32>, 8);
+  return go(head_norm_gate_kernel<S, 1>, 8);
 }
 
 }  // namespace

@@ -65,4 +65,23 @@ inline int make_rows_map(CUtensorMap* map, const void* base, int width, int n_ro
   return L3CI_OK;
 }
 
+// Rank-4 map over a [B, heads, rows, width] view of 2- or 4-byte floats, boxes of box_rows rows by box_width columns of one head,
+// not swizzled; what lies beyond the view reads as 0.  Strides in elements, whole 16-byte vectors.
+inline int make_box_map(CUtensorMap* map, const void* base, int elem_bytes, int width, int rows, int heads, int B, long long st, long long sh,
+                        long long sb, int box_width, int box_rows) {
+  auto enc = tensor_map_encoder();
+  if (!enc) return fail(L3CI_ERR_CUDA, "cuTensorMapEncodeTiled is not available");
+  const cuuint64_t any = ((cuuint64_t)width * elem_bytes + 15) / 16 * 16;   // a dimension of extent 1 may carry any stride
+  cuuint64_t dims[4] = {(cuuint64_t)width, (cuuint64_t)rows, (cuuint64_t)heads, (cuuint64_t)B};
+  cuuint64_t strides[3] = {rows > 1 ? (cuuint64_t)st * elem_bytes : any, heads > 1 ? (cuuint64_t)sh * elem_bytes : any,
+                           B > 1 ? (cuuint64_t)sb * elem_bytes : any};
+  cuuint32_t box[4] = {(cuuint32_t)box_width, (cuuint32_t)box_rows, 1u, 1u};
+  cuuint32_t estr[4] = {1u, 1u, 1u, 1u};
+  const CUresult r = enc(map, elem_bytes == 4 ? CU_TENSOR_MAP_DATA_TYPE_FLOAT32 : CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 4, const_cast<void*>(base),
+                         dims, strides, box, estr, CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_NONE,
+                         CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
+  if (r != CUDA_SUCCESS) return fail(L3CI_ERR_CUDA, "cuTensorMapEncodeTiled failed with %d", (int)r);
+  return L3CI_OK;
+}
+
 }  // namespace l3ci
