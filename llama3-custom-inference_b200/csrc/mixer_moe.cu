@@ -14,7 +14,7 @@
 namespace l3ci {
 namespace {
 
-constexpr int kRouteWarps = 8;
+constexpr int kRouteWarps = 8, kRouteWarpsMax = 32;
 
 // Order of the floats as unsigned numbers; NaN is below every number.
 __device__ __forceinline__ unsigned ordered(float z) {
@@ -22,12 +22,13 @@ __device__ __forceinline__ unsigned ordered(float z) {
   return z != z ? 0u : u & 0x80000000u ? ~u : u | 0x80000000u;
 }
 
-__global__ void __launch_bounds__(32 * kRouteWarps)
+__global__ void __launch_bounds__(32 * kRouteWarpsMax)
 moe_route_kernel(const float* __restrict__ logits, const float* __restrict__ bias, int* __restrict__ experts, int* __restrict__ ranks,
                  float* __restrict__ weights, int* __restrict__ counts, long long rows, int tokens, int E, int top) {
   extern __shared__ float sh[];
+  const int warps = blockDim.x / kWarp;
   float* row = sh;                                                // [warps][E]
-  int* count = reinterpret_cast<int*>(row + kRouteWarps * E);     // [E], then the expert's first rank of this CTA
+  int* count = reinterpret_cast<int*>(row + warps * E);           // [E], then the expert's first rank of this CTA
   int* chosen = count + E;                                        // [tokens][top]
   int* place = chosen + tokens * top;                             // [tokens][top]
   float* weight = reinterpret_cast<float*>(place + tokens * top);
@@ -39,7 +40,7 @@ moe_route_kernel(const float* __restrict__ logits, const float* __restrict__ bia
   const long long row0 = (long long)blockIdx.x * tokens;
   const int n = (int)min((long long)tokens, rows - row0);
   float* z = row + warp * E;
-  for (int t = warp; t < n; t += kRouteWarps) {
+  for (int t = warp; t < n; t += warps) {
     for (int e = lane; e < E; e += 32) z[e] = logits[(row0 + t) * E + e] + bias[e];
     __syncwarp();
     float first = 0.f, sum = 0.f;
@@ -70,8 +71,15 @@ moe_route_kernel(const float* __restrict__ logits, const float* __restrict__ bia
     for (int j = lane; j < top; j += 32) weights[(row0 + t) * top + j] = weight[t * top + j] / sum;
   }
   __syncthreads();
-  for (int e = tid; e < E; e += blockDim.x)
-    if (count[e] > 0) count[e] = atomicAdd(counts + e, count[e]);
+  if (gridDim.x == 1) {                                           // these are all the tokens there are
+    for (int e = tid; e < E; e += blockDim.x) {
+      counts[e] = count[e];
+      count[e] = 0;
+    }
+  } else {
+    for (int e = tid; e < E; e += blockDim.x)
+      if (count[e] > 0) count[e] = atomicAdd(counts + e, count[e]);
+  }
   __syncthreads();
   for (int i = tid; i < n * top; i += blockDim.x) {
     experts[row0 * top + i] = chosen[i];
@@ -193,15 +201,23 @@ int l3ci_moe_route(const float* logits, const float* bias, int32_t* experts, int
     return fail(L3CI_ERR_INVALID, "moe_route: rows=%lld experts=%d top=%d", (long long)rows, E, top);
   if (!counts) return fail(L3CI_ERR_INVALID, "moe_route: null pointer");
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream_);
-  L3CI_CUDA_TRY(cudaMemsetAsync(counts, 0, sizeof(int32_t) * E, s));
-  if (rows == 0) return L3CI_OK;
+  if (rows == 0) {
+    L3CI_CUDA_TRY(cudaMemsetAsync(counts, 0, sizeof(int32_t) * E, s));
+    return L3CI_OK;
+  }
   if (!logits || !bias || !experts || !ranks || !weights) return fail(L3CI_ERR_INVALID, "moe_route: null pointer");
+  // few tokens: one CTA, which needs no counting across CTAs
   const int sms = sm_count() > 0 ? sm_count() : 148;
-  int tokens = rows >= 16LL * sms ? 4 * kRouteWarps : rows >= kRouteWarps ? kRouteWarps : 1;
-  auto bytes = [&](int n) { return sizeof(float) * ((size_t)kRouteWarps * E + E + 3 * (size_t)n * top); };
-  while (tokens > 1 && bytes(tokens) > (48 << 10)) tokens /= 2;
-  if (bytes(tokens) > (48 << 10)) return fail(L3CI_ERR_UNSUPPORTED, "moe_route: experts=%d top=%d", E, top);
-  L3CI_LAUNCH("moe_route_kernel", moe_route_kernel, dim3((unsigned)((rows + tokens - 1) / tokens)), dim3(32 * kRouteWarps), bytes(tokens), s, logits,
+  auto bytes = [&](int warps, int n) { return sizeof(float) * ((size_t)warps * E + E + 3 * (size_t)n * top); };
+  int warps = (int)(rows < kRouteWarpsMax ? rows : kRouteWarpsMax), tokens = (int)(rows < 4 * kRouteWarpsMax ? rows : 4 * kRouteWarpsMax);
+  if (rows > tokens || bytes(warps, tokens) > (48 << 10)) {
+    warps = kRouteWarps;
+    tokens = rows >= 16LL * sms ? 4 * kRouteWarps : kRouteWarps;
+    while (tokens > 1 && bytes(warps, tokens) > (48 << 10)) tokens /= 2;
+    if (bytes(warps, tokens) > (48 << 10)) return fail(L3CI_ERR_UNSUPPORTED, "moe_route: experts=%d top=%d", E, top);
+  }
+  if (rows > tokens) L3CI_CUDA_TRY(cudaMemsetAsync(counts, 0, sizeof(int32_t) * E, s));
+  L3CI_LAUNCH("moe_route_kernel", moe_route_kernel, dim3((unsigned)((rows + tokens - 1) / tokens)), dim3(32 * warps), bytes(warps, tokens), s, logits,
               bias, experts, ranks, weights, counts, (long long)rows, tokens, E, top);
   return L3CI_OK;
 }

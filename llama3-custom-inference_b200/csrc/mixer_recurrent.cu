@@ -698,11 +698,11 @@ head_norm_gate_kernel(S* __restrict__ out, long long out_st, long long out_sh, c
 }
 
 // ---- inputs of the delta rule -----------------------------------------------------------------------------------
-constexpr int kRun = 8;            // consecutive tokens of a warp
+constexpr int kRun = 8;            // consecutive tokens of a warp (one token per sequence: 1)
 constexpr int kMaxTaps = 4;        // taps whose inputs stay in registers along the run
 
 // TAPS > 0: the run's inputs are all asked for at once and every one is loaded once; 0: any number of taps.
-template <typename S, int VEC, int TAPS>
+template <typename S, int VEC, int TAPS, int RUN>
 __global__ void __launch_bounds__(256) delta_inputs_kernel(const l3ci_delta_inputs_args a, int runs, long long tasks) {
   pdl_wait();
   pdl_launch_dependents();
@@ -713,7 +713,7 @@ __global__ void __launch_bounds__(256) delta_inputs_kernel(const l3ci_delta_inpu
   // neighbouring warps take neighbouring heads of the same tokens
   const int what = (int)(id % kinds);
   const long long run = id / kinds;
-  const int b = (int)(run / runs), t0 = (int)(run % runs) * kRun, n = min(kRun, a.T - t0);
+  const int b = (int)(run / runs), t0 = (int)(run % runs) * RUN, n = min(RUN, a.T - t0);
   const long long row0 = (long long)b * a.T;
   const int GD = a.G * a.D;
   const long long C_all = 2LL * GD + (long long)a.H * a.V;
@@ -726,19 +726,23 @@ __global__ void __launch_bounds__(256) delta_inputs_kernel(const l3ci_delta_inpu
       a.beta_out[(row0 + t0 + lane) * a.H + h] = sigmoid(z);
     }
     for (int c = lane * VEC; c < a.D; c += 32 * VEC) {
-      float z[kRun][VEC], bias[VEC];
+      using R = typename Raw<VEC * sizeof(S)>::type;
+      R raw[RUN];
+      float bias[VEC];
+#pragma unroll
+      for (int x = 0; x < RUN; ++x) raw[x] = *reinterpret_cast<const R*>(src + min(x, n - 1) * a.a_st + c);
       load_vec<float, VEC>(a.dt_bias + (long long)h * a.D + c, bias);
 #pragma unroll
-      for (int x = 0; x < kRun; ++x) load_vec<S, VEC>(src + min(x, n - 1) * a.a_st + c, z[x]);
-#pragma unroll
-      for (int x = 0; x < kRun; ++x) {
+      for (int x = 0; x < RUN; ++x) {
         if (x >= n) break;
+        float z[VEC];
+        load_vec<S, VEC>(reinterpret_cast<const S*>(&raw[x]), z);
 #pragma unroll
         for (int k = 0; k < VEC; ++k) {
-          const float y = z[x][k] + bias[k];
-          z[x][k] = expf(-rate * (fmaxf(y, 0.f) + log1pf(expf(-fabsf(y)))));
+          const float y = z[k] + bias[k];
+          z[k] = expf(-rate * (fmaxf(y, 0.f) + log1pf(expf(-fabsf(y)))));
         }
-        store_vec<float, VEC>(a.decay_out + ((row0 + t0 + x) * a.H + h) * a.D + c, z[x]);
+        store_vec<float, VEC>(a.decay_out + ((row0 + t0 + x) * a.H + h) * a.D + c, z);
       }
     }
     return;
@@ -779,13 +783,28 @@ __global__ void __launch_bounds__(256) delta_inputs_kernel(const l3ci_delta_inpu
     for (int c = lane * VEC; c < (is_v ? size : 32 * VEC); c += 32 * VEC) {    // (every lane takes part in a unit vector's sums)
       const bool mine = c < size;
       const int at = mine ? c : 0;
-      float f[kRun + kTaps - 1][VEC], w[kTaps][VEC];
+      using R = typename Raw<VEC * sizeof(S)>::type;
+      R raw[RUN + kTaps - 1];
+      float f[RUN + kTaps - 1][VEC], w[kTaps][VEC];
+      // (addresses chosen, not branches taken: every load is in flight before the first is used)
 #pragma unroll
-      for (int i = 0; i < kRun + kTaps - 1; ++i) input(min(t0 - (kTaps - 1) + i, a.T - 1), at, f[i]);
+      for (int i = 0; i < RUN + kTaps - 1; ++i) {
+        const int t = min(t0 - (kTaps - 1) + i, a.T - 1);
+        const S* from = t >= 0 || fresh ? in + (long long)max(t, 0) * a.p_st : tail + (kTaps - 1 + t) * C_all;
+        raw[i] = *reinterpret_cast<const R*>(from + at);
+      }
 #pragma unroll
       for (int i = 0; i < kTaps; ++i) load_vec<float, VEC>(a.conv + i * C_all + ch0 + at, w[i]);
 #pragma unroll
-      for (int x = 0; x < kRun; ++x) {
+      for (int i = 0; i < RUN + kTaps - 1; ++i) {
+        load_vec<S, VEC>(reinterpret_cast<const S*>(&raw[i]), f[i]);
+        if (i < kTaps - 1 && fresh && t0 - (kTaps - 1) + i < 0) {
+#pragma unroll
+          for (int k = 0; k < VEC; ++k) f[i][k] = 0.f;
+        }
+      }
+#pragma unroll
+      for (int x = 0; x < RUN; ++x) {
         if (x >= n) break;
         float y[VEC], ss = 0.f;
 #pragma unroll
@@ -964,7 +983,7 @@ int l3ci_delta_inputs(const l3ci_delta_inputs_args* a) {
   if (!a->p || !a->a || !a->b || !a->conv || !a->a_log || !a->dt_bias || (!a->tail && a->taps > 1) || !a->positions || !a->qk_out || !a->beta_out ||
       !a->decay_out || !a->v_out)
     return fail(L3CI_ERR_INVALID, "delta_inputs: null pointer");
-  const int runs = (a->T + kRun - 1) / kRun;
+  const int run = a->T == 1 ? 1 : kRun, runs = (a->T + run - 1) / run;
   const long long tasks = (long long)a->B * runs * (2 * a->G + 2 * a->H);
   if ((tasks + 7) / 8 > 0x7fffffffLL) return fail(L3CI_ERR_INVALID, "delta_inputs: too many rows");
   cudaStream_t s = reinterpret_cast<cudaStream_t>(a->stream);
@@ -974,18 +993,18 @@ int l3ci_delta_inputs(const l3ci_delta_inputs_args* a) {
     const int s4 = 4 * (int)sizeof(S);
     const bool v4 = (a->D | a->V | a->p_st | a->a_st | a->tail_sb) % 4 == 0 && on(a->p, s4) && on(a->a, s4) && on(a->tail, s4) && on(a->v_out, s4) &&
                     on(a->conv, 16) && on(a->dt_bias, 16) && on(a->qk_out, 16) && on(a->decay_out, 16);
-    auto go = [&](auto kernel) -> int {
-      L3CI_LAUNCH("delta_inputs_kernel", kernel, dim3((unsigned)((tasks + 7) / 8)), dim3(256), 0, s, *a, runs, tasks);
+    auto go = [&](auto one, auto many) -> int {
+      L3CI_LAUNCH("delta_inputs_kernel", run == 1 ? one : many, dim3((unsigned)((tasks + 7) / 8)), dim3(256), 0, s, *a, runs, tasks);
       return L3CI_OK;
     };
-    if (!v4) return go(delta_inputs_kernel<S, 1, 0>);
+    if (!v4) return go(delta_inputs_kernel<S, 1, 0, 1>, delta_inputs_kernel<S, 1, 0, kRun>);
     switch (a->taps) {
-      case 1: return go(delta_inputs_kernel<S, 4, 1>);
-      case 2: return go(delta_inputs_kernel<S, 4, 2>);
-      case 3: return go(delta_inputs_kernel<S, 4, 3>);
-      case kMaxTaps: return go(delta_inputs_kernel<S, 4, kMaxTaps>);
+      case 1: return go(delta_inputs_kernel<S, 4, 1, 1>, delta_inputs_kernel<S, 4, 1, kRun>);
+      case 2: return go(delta_inputs_kernel<S, 4, 2, 1>, delta_inputs_kernel<S, 4, 2, kRun>);
+      case 3: return go(delta_inputs_kernel<S, 4, 3, 1>, delta_inputs_kernel<S, 4, 3, kRun>);
+      case kMaxTaps: return go(delta_inputs_kernel<S, 4, kMaxTaps, 1>, delta_inputs_kernel<S, 4, kMaxTaps, kRun>);
     }
-    return go(delta_inputs_kernel<S, 4, 0>);
+    return go(delta_inputs_kernel<S, 4, 0, 1>, delta_inputs_kernel<S, 4, 0, kRun>);
   };
   return a->dtype == L3CI_BF16 ? typed(__nv_bfloat16{}) : typed(float{});
 }

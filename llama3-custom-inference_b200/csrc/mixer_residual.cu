@@ -21,7 +21,8 @@ namespace l3ci {
 namespace {
 
 constexpr int kMaxWarps = 16;
-constexpr int kManyVpt = 8;    // vectors of a thread when there are many rows
+constexpr int kManyVpt = 4;    // vectors of a thread when there are many rows
+constexpr int kPartsAhead = 4;
 
 // Mean and 1 / sqrt(variance + eps) of a row of `width` values; the thread's values are the first `valid` of v.
 template <int N>
@@ -59,8 +60,9 @@ __device__ __forceinline__ float sinusoid(int p, double freq, bool cosine) {
   return cosine ? cosf(angle) : sinf(angle);
 }
 
-template <typename S, int VEC, int VPT>
-__global__ void __launch_bounds__(VPT >= 16 ? 256 : 512) residual_norm_kernel(const l3ci_residual_norm_args a) {
+// Y: type of y.
+template <typename S, typename Y, int VEC, int VPT>
+__global__ void __launch_bounds__(512) residual_norm_kernel(const l3ci_residual_norm_args a) {
   __shared__ float sm[2][kMaxWarps][3];
   const int tid = threadIdx.x, width = (int)a.width;
   int col[VPT], chunks = 0;
@@ -107,17 +109,43 @@ __global__ void __launch_bounds__(VPT >= 16 ? 256 : 512) residual_norm_kernel(co
       }
     }
     if (a.y) {
-      for (int p = 0; p < a.parts; ++p) {
-        const float w = a.part_weights ? a.part_weights[row * a.parts + p] : 1.f;
-        const long long at = (a.part_rows ? a.part_rows[row * a.parts + p] : row * a.parts + p) * (long long)width;
+      const Y* ys = static_cast<const Y*>(a.y);
+      if (a.parts == 1 && !a.part_rows) {
+        const float w = a.part_weights ? a.part_weights[row] : 1.f;
 #pragma unroll
         for (int i = 0; i < VPT; ++i) {
           if (i >= chunks) break;
           float f[VEC];
-          if (a.y_dtype == L3CI_F32) load_vec<float, VEC>(static_cast<const float*>(a.y) + at + col[i], f);
-          else load_vec<__nv_bfloat16, VEC>(static_cast<const __nv_bfloat16*>(a.y) + at + col[i], f);
+          load_vec<Y, VEC>(ys + row * width + col[i], f);
 #pragma unroll
-          for (int k = 0; k < VEC; ++k) y[i * VEC + k] = fmaf(w, f[k], y[i * VEC + k]);
+          for (int k = 0; k < VEC; ++k) y[i * VEC + k] = w * f[k];
+        }
+      } else {
+        for (int p0 = 0; p0 < a.parts; p0 += kPartsAhead) {      // several parts' rows in flight
+          long long at[kPartsAhead];
+          float w[kPartsAhead];
+#pragma unroll
+          for (int p = 0; p < kPartsAhead; ++p) {
+            const long long id = row * a.parts + min(p0 + p, a.parts - 1);
+            at[p] = (a.part_rows ? a.part_rows[id] : id) * (long long)width;
+            w[p] = p0 + p >= a.parts ? 0.f : a.part_weights ? a.part_weights[id] : 1.f;
+          }
+#pragma unroll
+          for (int i = 0; i < VPT; ++i) {
+            if (i >= chunks) break;
+            using R = typename Raw<VEC * sizeof(Y)>::type;
+            R raw[kPartsAhead];
+#pragma unroll
+            for (int p = 0; p < kPartsAhead; ++p) raw[p] = *reinterpret_cast<const R*>(ys + at[p] + col[i]);
+#pragma unroll
+            for (int p = 0; p < kPartsAhead; ++p) {
+              if (p0 + p >= a.parts) break;
+              float f[VEC];
+              load_vec<Y, VEC>(reinterpret_cast<const Y*>(&raw[p]), f);
+#pragma unroll
+              for (int k = 0; k < VEC; ++k) y[i * VEC + k] = fmaf(w[p], f[k], y[i * VEC + k]);
+            }
+          }
         }
       }
       if (a.post_w) {
@@ -178,39 +206,35 @@ __global__ void __launch_bounds__(VPT >= 16 ? 256 : 512) residual_norm_kernel(co
   }
 }
 
-template <typename S>
+template <typename S, typename Y>
 int residual_norm_typed(const l3ci_residual_norm_args* a) {
-  auto ok = [](const void* p, int bytes) { return (reinterpret_cast<uintptr_t>(p) & (bytes - 1)) == 0; };
-  const int s4 = 4 * (int)sizeof(S);
-  const bool v4 = a->width % 4 == 0 && ok(a->x, 16) && ok(a->y, a->y_dtype == L3CI_F32 ? 16 : 8) && ok(a->post_w, 16) && ok(a->post_b, 16) &&
-                  ok(a->step, 16) && ok(a->pre_w, 16) && ok(a->pre_b, 16) && ok(a->out, s4) && a->out_stride % 4 == 0 && ok(a->table, s4) &&
-                  ok(a->x0, s4) && a->x0_stride % 4 == 0;
-  const long long units = v4 ? a->width / 4 : a->width;
+  constexpr int kVec = 8;
+  auto ok = [](const void* p) { return aligned16(p); };
+  const bool vec = a->width % kVec == 0 && ok(a->x) && ok(a->y) && ok(a->post_w) && ok(a->post_b) && ok(a->step) && ok(a->pre_w) && ok(a->pre_b) &&
+                   ok(a->out) && a->out_stride % kVec == 0 && ok(a->table) && ok(a->x0) && a->x0_stride % kVec == 0;
+  const long long units = vec ? a->width / kVec : a->width;
   // few rows: as many threads as there are vectors; many rows: few threads with many vectors each, so that little of the work
   // is reductions and many rows are on an SM
   const bool many = a->rows > 4LL * (sm_count() > 0 ? sm_count() : 148);
   int threads = 32, vpt = 1;
-  while ((many && v4 ? kManyVpt : 1) * threads < units && threads < 512) threads *= 2;
+  while ((many && vec ? kManyVpt : 1) * threads < units && threads < 512) threads *= 2;
   while ((long long)vpt * threads < units) vpt *= 2;
-  if (threads > (vpt >= 16 ? 256 : 512)) return fail(L3CI_ERR_UNSUPPORTED, "residual_norm: width %lld", (long long)a->width);
   auto go = [&](auto kernel) -> int {
     L3CI_LAUNCH("residual_norm_kernel", kernel, dim3((unsigned)a->rows), dim3(threads), 0, reinterpret_cast<cudaStream_t>(a->stream), *a);
     return L3CI_OK;
   };
-  if (v4) {
+  if (vec) {
     switch (vpt) {
-      case 1: return go(residual_norm_kernel<S, 4, 1>);
-      case 2: return go(residual_norm_kernel<S, 4, 2>);
-      case 4: return go(residual_norm_kernel<S, 4, 4>);
-      case 8: return go(residual_norm_kernel<S, 4, 8>);
-      case 16: return go(residual_norm_kernel<S, 4, 16>);
+      case 1: return go(residual_norm_kernel<S, Y, kVec, 1>);
+      case 2: return go(residual_norm_kernel<S, Y, kVec, 2>);
+      case 4: return go(residual_norm_kernel<S, Y, kVec, 4>);
     }
   } else {
     switch (vpt) {
-      case 1: return go(residual_norm_kernel<S, 1, 1>);
-      case 2: return go(residual_norm_kernel<S, 1, 2>);
-      case 4: return go(residual_norm_kernel<S, 1, 4>);
-      case 8: return go(residual_norm_kernel<S, 1, 8>);
+      case 1: return go(residual_norm_kernel<S, Y, 1, 1>);
+      case 2: return go(residual_norm_kernel<S, Y, 1, 2>);
+      case 4: return go(residual_norm_kernel<S, Y, 1, 4>);
+      case 8: return go(residual_norm_kernel<S, Y, 1, 8>);
     }
   }
   return fail(L3CI_ERR_UNSUPPORTED, "residual_norm: width %lld", (long long)a->width);
@@ -231,5 +255,7 @@ extern "C" int l3ci_residual_norm(const l3ci_residual_norm_args* a) {
   if (!a->x || (!a->post_w) != (!a->post_b) || (!a->pre_w) != (!a->pre_b) || (a->reset && !a->y) ||
       (a->tokens && (!a->table || !a->positions || a->T <= 0 || a->vocab <= 0 || a->y)))
     return fail(L3CI_ERR_INVALID, "residual_norm: null pointer, or both y and tokens");
-  return a->dtype == L3CI_BF16 ? residual_norm_typed<__nv_bfloat16>(a) : residual_norm_typed<float>(a);
+  const bool y32 = a->y && a->y_dtype == L3CI_F32;
+  if (a->dtype == L3CI_F32) return y32 || !a->y ? residual_norm_typed<float, float>(a) : residual_norm_typed<float, __nv_bfloat16>(a);
+  return y32 ? residual_norm_typed<__nv_bfloat16, float>(a) : residual_norm_typed<__nv_bfloat16, __nv_bfloat16>(a);
 }
