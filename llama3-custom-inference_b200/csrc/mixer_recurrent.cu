@@ -701,9 +701,22 @@ head_norm_gate_kernel(S* __restrict__ out, long long out_st, long long out_sh, c
 constexpr int kRun = 8;            // consecutive tokens of a warp (one token per sequence: 1)
 constexpr int kMaxTaps = 4;        // taps whose inputs stay in registers along the run
 
+// exp(-rate * softplus(y)).  For bf16 models (y itself carries a bf16 rounding) with the short forms of exp and log; log1p(e) by
+// its series where 1 + e would round e away.
+template <typename S>
+__device__ __forceinline__ float decay_of(float y, float rate) {
+  if constexpr (sizeof(S) == 4) {
+    return expf(-rate * (fmaxf(y, 0.f) + log1pf(expf(-fabsf(y)))));
+  } else {
+    const float e = __expf(-fabsf(y));
+    const float l = e > 0.01f ? __logf(1.f + e) : e * fmaf(e, fmaf(e, 0.33333333f, -0.5f), 1.f);
+    return __expf(-rate * (fmaxf(y, 0.f) + l));
+  }
+}
+
 // TAPS > 0: the run's inputs are all asked for at once and every one is loaded once; 0: any number of taps.
 template <typename S, int VEC, int TAPS, int RUN>
-__global__ void __launch_bounds__(256) delta_inputs_kernel(const l3ci_delta_inputs_args a, int runs, long long tasks) {
+__global__ void __launch_bounds__(256, 3) delta_inputs_kernel(const l3ci_delta_inputs_args a, int runs, long long tasks) {
   pdl_wait();
   pdl_launch_dependents();
   const int lane = threadIdx.x & 31;
@@ -739,8 +752,7 @@ __global__ void __launch_bounds__(256) delta_inputs_kernel(const l3ci_delta_inpu
         load_vec<S, VEC>(reinterpret_cast<const S*>(&raw[x]), z);
 #pragma unroll
         for (int k = 0; k < VEC; ++k) {
-          const float y = z[k] + bias[k];
-          z[k] = expf(-rate * (fmaxf(y, 0.f) + log1pf(expf(-fabsf(y)))));
+          z[k] = decay_of<S>(z[k] + bias[k], rate);
         }
         store_vec<float, VEC>(a.decay_out + ((row0 + t0 + x) * a.H + h) * a.D + c, z);
       }
@@ -777,7 +789,8 @@ __global__ void __launch_bounds__(256) delta_inputs_kernel(const l3ci_delta_inpu
     if (is_v) store_vec<S, VEC>(static_cast<S*>(a.v_out) + row * a.H * a.V + (long long)(what - 2 * a.G) * a.V + c, r);
     else store_vec<float, VEC>(a.qk_out + row * 2 * GD + ch0 + c, r);
   };
-  auto unit = [&](float ss) { return is_v ? 1.f : 1.f / sqrtf(ss + a.unit_eps) / (what < a.G ? sqrtf((float)a.D) : 1.f); };
+  const float length = what < a.G ? rsqrtf((float)a.D) : 1.f;
+  auto unit = [&](float ss) { return is_v ? 1.f : rsqrtf(ss + a.unit_eps) * length; };
   if (TAPS > 0 && (is_v || size <= 32 * VEC)) {
     constexpr int kTaps = TAPS > 0 ? TAPS : 1;
     for (int c = lane * VEC; c < (is_v ? size : 32 * VEC); c += 32 * VEC) {    // (every lane takes part in a unit vector's sums)

@@ -21,7 +21,7 @@ namespace l3ci {
 namespace {
 
 constexpr int kMaxWarps = 16;
-constexpr int kManyVpt = 4;    // vectors of a thread when there are many rows
+constexpr int kManyVpt = 2;    // vectors of a thread when there are many rows
 constexpr int kPartsAhead = 4;
 
 // Mean and 1 / sqrt(variance + eps) of a row of `width` values; the thread's values are the first `valid` of v.
