@@ -1217,7 +1217,8 @@ class KernelTable:
 
 def rupotar_kernel_table(ext, pkg, dev, cfg):
     """Every kernel of the Rupotar decoder beside the kernel of the Nibelorn decoder that does the like.  Bytes: inputs and
-    outputs once; the scans over prompts against the fp32 rate of the device (`fma`), which is what they run on."""
+    outputs once; the scans over prompts against the fp32 rate of the device (`fma`), which is what they run on, with the
+    operations of the recurrence itself (delta rule: decay, S^T k, the write, S^T q; time mixing: decay, write, S^T r)."""
     ru, mx, tab = pkg.rupotar, pkg.mixers, KernelTable(dev)
     us, sets, row, byte, flop = tab.us, tab.sets, tab.row, tab.byte, tab.flop
     fma = torch.cuda.get_device_properties(dev).multi_processor_count * 128 * 2 * 1.965e3      # fp32 flops per microsecond at the top clock
