@@ -42,9 +42,9 @@ constexpr int kMaxConsumers[2] = {8, 16};   // warps, by kind
 constexpr int kHelpers[2] = {1, 2};   // warps, by kind
 // A warp's patch of output shares: 32 / C tokens of 32 lanes of C floats, tokens a little apart (no bank conflicts).
 template <int C>
-constexpr int kPatchToken = 32 * C + (C == 4 ? 16 : 32);   // floats
+constexpr int kPatchToken = 32 * C + (C == 2 ? 4 : C == 4 ? 16 : 32);   // floats
 constexpr int kPatchBytes = 8 * kPatchToken<4> * 4;
-static_assert(kPatchBytes >= 4 * kPatchToken<8> * 4, "a patch holds either form");
+static_assert(kPatchBytes >= 4 * kPatchToken<8> * 4 && kPatchBytes >= 16 * kPatchToken<2> * 4, "a patch holds every form");
 
 __device__ __forceinline__ float sigmoid(float z) { return 1.f / (1.f + expf(-z)); }
 __device__ __forceinline__ float gate_value(float z, int act) { return act == 0 ? sigmoid(z) : z * sigmoid(z); }
@@ -92,6 +92,29 @@ __device__ __forceinline__ void load_rows(const Q* p, int lane, unsigned long lo
         r[i * (W / 2) + e] = f2_packf(bf16lo_to_f32(x), bf16hi_to_f32(x));
       }
     }
+  }
+}
+// N neighbouring fp32 columns (2, or a multiple of 4).
+template <int N>
+__device__ __forceinline__ void load_cols(const float* p, float* f) {
+  if constexpr (N == 2) {
+    const float2 x = *reinterpret_cast<const float2*>(p);
+    f[0] = x.x; f[1] = x.y;
+  } else {
+#pragma unroll
+    for (int c = 0; c < N; c += 4) {
+      const float4 x = *reinterpret_cast<const float4*>(p + c);
+      f[c] = x.x; f[c + 1] = x.y; f[c + 2] = x.z; f[c + 3] = x.w;
+    }
+  }
+}
+template <int N>
+__device__ __forceinline__ void store_cols(float* p, const float* f) {
+  if constexpr (N == 2) {
+    *reinterpret_cast<float2*>(p) = make_float2(f[0], f[1]);
+  } else {
+#pragma unroll
+    for (int c = 0; c < N; c += 4) *reinterpret_cast<float4*>(p + c) = make_float4(f[c], f[c + 1], f[c + 2], f[c + 3]);
   }
 }
 template <int N>
@@ -309,11 +332,7 @@ recurrent_scan_kernel(const __grid_constant__ CUtensorMap qmap, const __grid_con
       if (fresh || row >= D) continue;
       const float* at = state + (long long)row * V;
       if (wide) {
-#pragma unroll
-        for (int c = 0; c < C; c += 4) {
-          const float4 x = *reinterpret_cast<const float4*>(at + c);
-          f[e][c] = x.x; f[e][c + 1] = x.y; f[e][c + 2] = x.z; f[e][c + 3] = x.w;
-        }
+        load_cols<C>(at, f[e]);
       } else {
 #pragma unroll
         for (int c = 0; c < C; ++c)
@@ -342,14 +361,15 @@ recurrent_scan_kernel(const __grid_constant__ CUtensorMap qmap, const __grid_con
   float* patch = reinterpret_cast<float*>(smem + ring * stage_bytes + 3 * kMaxRing * 8 + warp * kPatchBytes);
   // (stored behind the block's last token: between the tokens the stores would hold up the loads of the next one)
   auto share = [&](int x, const float* part) {
+    constexpr int kV = C < 4 ? C : 4;
 #pragma unroll
-    for (int c = 0; c < C; c += 4)
-      *reinterpret_cast<float4*>(patch + x * kPatchToken<C> + c / 4 * 128 + lane * 4) = make_float4(part[c], part[c + 1], part[c + 2], part[c + 3]);
+    for (int c = 0; c < C; c += kV) store_cols<kV>(patch + x * kPatchToken<C> + c * 32 + lane * kV, part + c);
   };
   // the outputs of the block's n tokens from t0 on: C lanes per token sum the shares of 32 / C lanes each, all columns, and
   // then halve the columns among themselves
   auto write = [&](int t0, int n) {
     __syncwarp();
+    constexpr int kV = C < 4 ? C : 4;
     const int x = lane / C, part = lane % C;
     float sums[C];
 #pragma unroll
@@ -357,9 +377,11 @@ recurrent_scan_kernel(const __grid_constant__ CUtensorMap qmap, const __grid_con
 #pragma unroll
     for (int i = 0; i < 32 / C; ++i)
 #pragma unroll
-      for (int c = 0; c < C; c += 4) {
-        const float4 y = *reinterpret_cast<const float4*>(patch + x * kPatchToken<C> + c / 4 * 128 + (i * C + part) * 4);
-        sums[c] += y.x; sums[c + 1] += y.y; sums[c + 2] += y.z; sums[c + 3] += y.w;
+      for (int c = 0; c < C; c += kV) {
+        float y[kV];
+        load_cols<kV>(patch + x * kPatchToken<C> + c * 32 + (i * C + part) * kV, y);
+#pragma unroll
+        for (int k = 0; k < kV; ++k) sums[c + k] += y[k];
       }
 #pragma unroll
     for (int m = C / 2; m >= 1; m /= 2) {
@@ -421,8 +443,7 @@ recurrent_scan_kernel(const __grid_constant__ CUtensorMap qmap, const __grid_con
 #pragma unroll
       for (int j = 0; j < NR / 2; ++j) qb[j] = f2_mul(f2_mul(q[j], bonus[j]), k[j]);
       float v[C];
-      load_vec<S, 4>(vs, reinterpret_cast<float(&)[4]>(v[0]));
-      if constexpr (C == 8) load_vec<S, 4>(vs + 4, reinterpret_cast<float(&)[4]>(v[4]));
+      load_vec<S, C>(vs, v);
 #pragma unroll
       for (int c = 0; c < C; ++c) {
         const unsigned long long v2 = f2_packf(v[c], v[c]);
@@ -491,8 +512,7 @@ recurrent_scan_kernel(const __grid_constant__ CUtensorMap qmap, const __grid_con
       if (row >= D) continue;
       float* at = state + (long long)row * V;
       if (wide) {
-#pragma unroll
-        for (int c = 0; c < C; c += 4) *reinterpret_cast<float4*>(at + c) = make_float4(f[e][c], f[e][c + 1], f[e][c + 2], f[e][c + 3]);
+        store_cols<C>(at, f[e]);
       } else {
 #pragma unroll
         for (int c = 0; c < C; ++c)
@@ -941,7 +961,7 @@ int scan_typed(const l3ci_recurrent_scan_args* a, cudaStream_t stream) {
            rows16(a->v, sizeof(S), a->v_st, a->v_sh);
   // columns per warp and warps per CTA: as many as leave enough CTAs for the device
   // (the delta rule wants the registers, time mixing the warps)
-  const struct { int C, W; } by_kind[2][4] = {{{8, 8}, {8, 4}, {4, 4}, {4, 2}}, {{4, 16}, {4, 8}, {4, 4}, {4, 2}}};
+  const struct { int C, W; } by_kind[2][4] = {{{8, 8}, {8, 4}, {2, 8}, {2, 4}}, {{4, 16}, {4, 8}, {2, 8}, {2, 4}}};
   int C = 4;
   for (const auto& s : by_kind[KIND]) {
     C = s.C;
@@ -958,8 +978,7 @@ int scan_typed(const l3ci_recurrent_scan_args* a, cudaStream_t stream) {
     return a->D <= 64 ? launch_scan<S, Q, KIND, 2, CC>(p, stream) : a->D <= 128 ? launch_scan<S, Q, KIND, 4, CC>(p, stream)
                                                                               : launch_scan<S, Q, KIND, 8, CC>(p, stream);
   };
-  if constexpr (KIND == kDelta) st = C == 8 ? by_rows(std::integral_constant<int, 8>{}) : by_rows(std::integral_constant<int, 4>{});
-  else st = by_rows(std::integral_constant<int, 4>{});
+  st = C == 2 ? by_rows(std::integral_constant<int, 2>{}) : by_rows(std::integral_constant<int, KIND == kDelta ? 8 : 4>{});
   if (st) return st;
   // norm and gate of the rows the scan has written
   const long long units = heads * a->T;
