@@ -1173,9 +1173,9 @@ def bench_rupotar(args, ext, pkg, dev, rank, world):
                    "global_batch": 64 * world, "seq_len": 1024, "parallelism": "replicas x%d" % world,
                    "l2": "weights and cache of a step exceed L2"},
         "kernels": rupotar_kernel_table(ext, pkg, dev, cfg) if rank == 0 else None,
-        # per step: embedding, token choice; per run two norms; per attention two, delta three, time mixing three (token shift, tanh,
-        # scan); per dense one, experts four; per pass of the loop one more norm
-        "gpu_launches": line["steps"] * (2 + 16 * 2 + 8 * 2 + 4 * 3 + 4 * 3 + 8 * 1 + 8 * 4 + 2),
+        # per step: embedding, token choice; per run two norms; per attention two (split merges on top), delta two, time mixing three
+        # (token shift, tanh, step); per dense one, experts four; per pass of the loop one more norm
+        "gpu_launches": line["steps"] * (2 + 16 * 2 + 8 * 2 + 4 * 2 + 4 * 3 + 8 * 1 + 8 * 4 + 2),
     }
 
 
